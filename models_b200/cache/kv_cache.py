@@ -21,7 +21,7 @@ by the caller-provided `allocate` function.
 
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 from typing import Callable, Dict, List, Optional, Sequence, Tuple
 
 from .pages import CacheFull, FreeList
@@ -148,6 +148,7 @@ class KvCache:
         for run, request in enumerate(requests):
             if request is None or cache_from[run] is not None:
                 continue
+            request = self._widest(request, [requests[r] for r, source in enumerate(cache_from) if source == run])
             group = by_key.get(request)
             if group is None:
                 group = CacheGroup(request, [], self.pages_for(request, max_step_tokens), page_size)
@@ -171,6 +172,14 @@ class KvCache:
             self.run_location[run] = self.run_location[source]
 
     # ---------------------------------------------------------------- storage
+
+    @staticmethod
+    def _widest(request: KvRequest, readers: Sequence[Optional[KvRequest]]) -> KvRequest:
+        """What a run must keep for itself and for the runs that read its storage: the widest window (no window at all if one
+        of them sees every position) and the most first positions."""
+        everyone = [request] + [r for r in readers if r is not None]
+        windows = [r.window for r in everyone]
+        return replace(request, window=None if None in windows else max(windows), keep_first=max(r.keep_first for r in everyone))
 
     def pages_for(self, request: KvRequest, max_step_tokens: Optional[int]) -> int:
         """Usable pages of the group of `request`."""

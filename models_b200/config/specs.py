@@ -288,7 +288,15 @@ class LatentAttentionSpec:
     """Causal softmax attention whose keys and values are expanded from ONE cached row per position:
     c = rmsnorm(down . xn) of `latent_dim` numbers (gain, eps `eps`); head h has k = up_k[h] . c (`head_dim`) and
     v = up_v[h] . c (`value_dim`); score = scale * q.k; no positions enter.  `gated`: head h's result is multiplied
-    by sigmoid(gate_h . xn), one number per head and token."""
+    by sigmoid(gate_h . xn), one number per head and token.
+
+    Variations.  `query_latent` n > 0: queries come from a latent of their own, q = up_q . rmsnorm(down_q . xn) of n numbers
+    (gain `weights["down_q_norm"]`, eps `eps`).  `position`: a query head has rotary_dim more coordinates behind its head_dim, and
+    `down` has rotary_dim more rows, one key part that all heads share; both are rotated over all of these coordinates by their
+    position, and the score is scale * (q.k + q_rotated.k_rotated); the rotated part is cached behind the latent.  `window` n: a
+    query sees itself and the n - 1 positions before it.  `gate_kind` "element": the heads side by side are multiplied element by
+    element by sigmoid(gate . xn).  `own_rows` False: the layer has no `down`; it reads the rows another run cached (the schedule
+    names it), with its own up_k, up_v, queries and window."""
 
     hidden_size: int
     num_heads: int
@@ -300,6 +308,11 @@ class LatentAttentionSpec:
     gated: bool
     weights: Mapping[str, str] = field(default_factory=dict, hash=False, compare=False)
     kind: str = "latent_attention"
+    query_latent: int = 0
+    position: Optional[RopeSpec] = None
+    window: Optional[int] = None
+    gate_kind: str = "head"
+    own_rows: bool = True
 
 
 @dataclass(frozen=True)
@@ -402,6 +415,8 @@ class RoutedFeedForwardSpec:
     # `keep_groups` best groups can be chosen; the weights are `weight_scale` times the chosen outputs' s, not renormalised.
     # `identity_experts` n: the router has num_experts + n outputs, the last n of which stand for experts without tensors
     # whose result is their input.  `shared_gated` False: the shared expert is added as it is (no `shared_gate_score` tensor).
+    # `rule` "table": there is no router; an integer tensor [vocab_size, top] (`weights["table"]`) gives every token id its
+    # experts, each with the weight 1 / top.
     rule: str = "top_logits"
     correction: bool = False
     groups: int = 1
@@ -409,6 +424,7 @@ class RoutedFeedForwardSpec:
     weight_scale: float = 1.0
     identity_experts: int = 0
     shared_gated: bool = True
+    vocab_size: int = 0
 
 
 @dataclass(frozen=True)
@@ -515,3 +531,66 @@ class OutputNormBlockSpec:
     feed_forward_norm: Optional[object]
     weights: Mapping[str, str] = field(default_factory=dict, hash=False, compare=False)
     kind: str = "output_norm"
+
+
+@dataclass(frozen=True)
+class DynamicTanhSpec:
+    """tanh(alpha * x) * weight + bias, element by element: a norm that computes no mean and no variance.  alpha is one number
+    (`weights`: alpha, weight, bias)."""
+
+    size: int
+    weights: Mapping[str, str] = field(default_factory=dict, hash=False, compare=False)
+    kind: str = "dynamic_tanh"
+
+
+@dataclass(frozen=True)
+class StateSpaceSpec:
+    """A state-space recurrence with one decay per head and token.  in . xn is laid out [z: inner | x: inner | B: groups * state |
+    C: groups * state | dt: heads], inner = heads * value_dim.  x, B and C together pass a short causal convolution per channel
+    (`conv_taps` weights, the last one meeting the current token, zeros before the start) with a bias, and a silu;
+    dt = softplus(dt + dt_bias).  Per head (head h uses group h / (heads / groups)), with a float32 state S [state, value_dim] that
+    starts at zero: S <- exp(-exp(A_log) dt) S + dt B x^T; y = S^T C + D x.  The heads side by side are multiplied by silu(z), then
+    divided by their root mean square in `norm_groups` equal parts (eps `eps`), times a gain; then the output matrix.  The last
+    conv_taps - 1 inputs of the convolution are part of the state."""
+
+    hidden_size: int
+    num_heads: int
+    value_dim: int
+    state_size: int
+    groups: int
+    norm_groups: int
+    conv_taps: int
+    eps: float
+    weights: Mapping[str, str] = field(default_factory=dict, hash=False, compare=False)
+    kind: str = "state_space"
+
+
+@dataclass(frozen=True)
+class TokenSideSpec:
+    """The token itself let in once more beside the stream: proj . (gelu_tanh(gate . x) * e), e = columns
+    [index * dim, (index + 1) * dim) of the token's row of a table [vocab_size, layers * dim] (`weights`: table, gate, proj)."""
+
+    hidden_size: int
+    vocab_size: int
+    dim: int
+    index: int
+    layers: int
+    weights: Mapping[str, str] = field(default_factory=dict, hash=False, compare=False)
+    kind: str = "token_side"
+
+
+@dataclass(frozen=True)
+class SandwichBlockSpec:
+    """A layer with a norm before and after each sublayer: x += mixer_out_norm(mixer(mixer_norm(x))); then, if the layer has a
+    feed-forward, x += feed_forward_out_norm(feed_forward(feed_forward_norm(x))); then, if it has a side input,
+    x += side_norm(side(x))."""
+
+    mixer: object
+    mixer_norm: object
+    mixer_out_norm: object
+    feed_forward: Optional[object] = None
+    feed_forward_norm: Optional[object] = None
+    feed_forward_out_norm: Optional[object] = None
+    side: Optional[object] = None
+    side_norm: Optional[object] = None
+    kind: str = "sandwich"

@@ -12,7 +12,7 @@
 // value in the softmax's denominator, p_j = exp(s_j) / (1 + sum exp(s_j)); and values that were stored rotated by their
 // own position (pairs 2m, 2m + 1): the head's sum is then turned back by the query's position before any gate.
 // Visibility may be cut into blocks: with `block` n > 0, query i sees key j <= i only if floor(i / n) = floor(j / n)
-// (blocks of n positions counted from position 0 of the sequence).
+// (blocks of n positions counted from position 0 of the sequence); with `window` n > 0, only if i - j < n.
 //
 // Keys have head_dim coordinates and values value_dim; the value rows may lie in a pool of their own or be the
 // first value_dim coordinates of the key rows (a cache that keeps one row per position, read as key and as value).
@@ -40,10 +40,14 @@ struct ScoreExtras {
     const float* turn_cos;    // [positions][value_dim / 2] with turn_sin: the result's pairs (2m, 2m + 1) are turned by
     const float* turn_sin;    // minus the query's position; null: the result stays as it is
     int block;                // n > 0: a query sees only the keys of its own block of n positions; 0: every earlier key
+    int window;               // n > 0: a query sees only itself and the n - 1 positions before it
 };
 
 // the first position a query at `pos` sees
-__device__ __forceinline__ int lowest_visible(int pos, int block) { return block > 0 ? (pos / block) * block : 0; }
+__device__ __forceinline__ int lowest_visible(int pos, const ScoreExtras& extras) {
+    const int of_block = extras.block > 0 ? (pos / extras.block) * extras.block : 0;
+    return extras.window > 0 ? max(of_block, pos - extras.window + 1) : of_block;
+}
 
 __device__ __forceinline__ float bounded(float z, float cap) { return cap > 0.0f ? cap * tanhf(z / cap) : z; }
 
@@ -341,6 +345,53 @@ __global__ void project_norm_rotate_store_kernel(T* __restrict__ q, int q_stride
     }
 }
 
+// grid (tokens); block 128.  What a latent attention does to the rows of its first product: the query's latent (q_width numbers,
+// null: none) divided by its root mean square and multiplied by its gain, into rows of its own that are zero up to q_columns;
+// and the row the cache keeps, [latent | tail]: the latent normalised the same way with its own gain, the tail's `turned`
+// numbers rotated by the token's position (pairs (i, i + turned / 2), tables [positions][turned / 2]).  k null: no row is stored.
+template <typename T>
+__global__ void __launch_bounds__(128)
+latent_prepare_kernel(const T* __restrict__ q, int q_stride, const float* __restrict__ q_gain, int q_width, T* __restrict__ q_out,
+                      int q_columns, const T* __restrict__ k, int k_stride, const float* __restrict__ k_gain, int latent, int turned,
+                      const float* __restrict__ cos, const float* __restrict__ sin, const int* __restrict__ positions, float eps,
+                      T* __restrict__ k_pool, const int* __restrict__ slot_mapping) {
+    grid_launch_dependents();
+    grid_dependency_wait();
+    __shared__ float scratch[32];
+    const size_t token = blockIdx.x;
+    if (q != nullptr) {
+        const T* src = q + token * q_stride;
+        float squares = 0.0f;
+        for (int i = threadIdx.x; i < q_width; i += blockDim.x) {
+            const float x = Num<T>::load(src + i);
+            squares = fmaf(x, x, squares);
+        }
+        const float factor = 1.0f / sqrtf(block_sum(squares, scratch) / (float)q_width + eps);
+        for (int i = threadIdx.x; i < q_columns; i += blockDim.x)
+            Num<T>::store(q_out + token * q_columns + i, i < q_width ? Num<T>::load(src + i) * factor * q_gain[i] : 0.0f);
+    }
+    if (k == nullptr) return;
+    const int slot = slot_mapping[token];
+    if (slot < 0) return;  // (the whole block) a padding row stores nothing
+    const T* src = k + token * k_stride;
+    T* dst = k_pool + (size_t)slot * (latent + turned);  // [page][1][page_size][latent + turned]: the slot counts rows
+    float squares = 0.0f;
+    for (int i = threadIdx.x; i < latent; i += blockDim.x) {
+        const float x = Num<T>::load(src + i);
+        squares = fmaf(x, x, squares);
+    }
+    const float factor = 1.0f / sqrtf(block_sum(squares, scratch) / (float)latent + eps);
+    for (int i = threadIdx.x; i < latent; i += blockDim.x) Num<T>::store(dst + i, Num<T>::load(src + i) * factor * k_gain[i]);
+    const int half = turned / 2;
+    const size_t row = half > 0 ? (size_t)positions[token] * half : 0;
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        const float c = cos[row + i], s = sin[row + i];
+        const float u = Num<T>::load(src + latent + i), v = Num<T>::load(src + latent + half + i);
+        Num<T>::store(dst + latent + i, u * c - v * s);
+        Num<T>::store(dst + latent + half + i, v * c + u * s);
+    }
+}
+
 template <typename T>
 __device__ __forceinline__ float dot_row(const float* __restrict__ q_shared, const T* __restrict__ k_row, int head_dim,
                                          bool vector_ok) {
@@ -398,7 +449,7 @@ gated_attention_rows_kernel(const T* __restrict__ q, int q_stride, T* __restrict
     float running_max = kSoftmax && extras.sink ? 0.0f : -CUDART_INF_F, running_sum = kSoftmax && extras.sink ? 1.0f : 0.0f;
     const int* table = block_table + (size_t)seq * max_blocks;
 
-    const int lowest = lowest_visible(pos, extras.block);
+    const int lowest = lowest_visible(pos, extras);
     for (int chunk = lowest & ~31; chunk <= pos; chunk += 32) {  // (the first chunk holds `lowest`: every chunk has a visible key)
         // page_size is a multiple of 32, so a chunk of 32 positions lies in one page
         const size_t page = table[chunk / page_size];
@@ -485,9 +536,10 @@ gated_attention_decode_kernel(const T* __restrict__ q, int q_stride, const T* __
     const int head0 = kv_head * group + part * kGroup;
     const int count = min(kGroup, group - part * kGroup);
     const int pos = kv_lens[seq] - 1;
-    const int lowest = lowest_visible(pos, extras.block);
-    const int end = min(pos + 1, (split + 1) * span * page_size);
-    const int begin = max(split * span * page_size, lowest & ~31);  // (the chunk of 32 that holds `lowest`: every chunk has a visible key)
+    const int lowest = lowest_visible(pos, extras);
+    const int first_page = lowest / page_size;  // the runs are counted from the first page that holds a visible key
+    const int end = min(pos + 1, (first_page + (split + 1) * span) * page_size);
+    const int begin = max((first_page + split * span) * page_size, lowest & ~31);  // (the chunk of 32 that holds `lowest`: every chunk has a visible key)
     const int stride = 2 + value_dim;
     float* q_shared = decode_shared;
     float* meet = decode_shared + kGroup * head_dim;  // [warp][kGroup][stride]
@@ -693,8 +745,28 @@ __global__ void gated_attention_combine_kernel(const float* __restrict__ partial
     Num<T>::store(out + row * out_stride + (size_t)head * value_dim + d, value);
 }
 
-// out[t, h * n_out + n] = gate * sum_k in[t, h * n_in + k] * w[(h * n_out + n) * n_in + k]: one small matrix per head,
-// rows of n_in weights; gate: sigmoid of gate[t, h] when given.
+// out[t, h * out_head + n] = gate * sum_k in[t, h * in_head + k] * w[(h * n_out + n) * n_in + k]: one small matrix per head,
+// rows of n_in weights; gate: sigmoid of gate[t, h], or of gate[t, h * n_out + n] when gates are per element (HeadLayout).
+// A head may have a tail of `turned` coordinates behind its n_in inputs that passes by the matrix: it is rotated by the token's
+// position (pairs (i, i + turned / 2), tables [positions][turned / 2]) and stored behind the head's n_out outputs.
+struct HeadLayout {
+    int in_head, out_head;  // elements from one head's inputs (outputs) to the next's
+    int element_gate;       // gate: one number per output instead of one per head
+    int turned;             // 0: no tail
+    const float* cos;
+    const float* sin;
+    const int* positions;
+};
+
+template <typename T>
+__device__ __forceinline__ void turn_tail(const T* __restrict__ src, T* __restrict__ dst, int pair, const HeadLayout& layout, int position) {
+    const int half = layout.turned / 2;
+    const float c = layout.cos[(size_t)position * half + pair], s = layout.sin[(size_t)position * half + pair];
+    const float u = Num<T>::load(src + pair), v = Num<T>::load(src + pair + half);
+    Num<T>::store(dst + pair, u * c - v * s);
+    Num<T>::store(dst + pair + half, v * c + u * s);
+}
+
 // Plain arithmetic: grid (ceil(tokens / 16), heads, ceil(n_out / 8)); block 128.  A warp takes 2 of the block's 8
 // outputs in turn (few, so that a decode step's handful of tokens still spreads over the multiprocessors and no warp
 // waits for memory many times in a row): its lanes walk a weight row together (neighbouring lanes read neighbouring
@@ -704,7 +776,8 @@ constexpr int kHeadOutputs = 8;
 
 template <typename T>
 __global__ void head_linear_kernel(const T* __restrict__ in, int in_stride, const T* __restrict__ w, T* __restrict__ out,
-                                   int out_stride, const T* __restrict__ gate, int gate_stride, int tokens, int n_in, int n_out) {
+                                   int out_stride, const T* __restrict__ gate, int gate_stride, int tokens, int n_in, int n_out,
+                                   HeadLayout layout) {
     grid_launch_dependents();
     grid_dependency_wait();
     extern __shared__ float rows_shared[];  // [kHeadRows][n_in]
@@ -713,7 +786,15 @@ __global__ void head_linear_kernel(const T* __restrict__ in, int in_stride, cons
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     for (int item = threadIdx.x; item < kHeadRows * n_in; item += blockDim.x) {
         const int r = item / n_in, k = item % n_in;
-        rows_shared[item] = r < rows ? Num<T>::load(in + (size_t)(first + r) * in_stride + (size_t)head * n_in + k) : 0.0f;
+        rows_shared[item] = r < rows ? Num<T>::load(in + (size_t)(first + r) * in_stride + (size_t)head * layout.in_head + k) : 0.0f;
+    }
+    if (layout.turned > 0 && blockIdx.z == 0) {
+        const int half = layout.turned / 2;
+        for (int item = threadIdx.x; item < rows * half; item += blockDim.x) {
+            const size_t row = first + item / half;
+            turn_tail<T>(in + row * in_stride + (size_t)head * layout.in_head + n_in, out + row * out_stride + (size_t)head * layout.out_head + n_out,
+                         item % half, layout, layout.positions[row]);
+        }
     }
     __syncthreads();
     for (int i = 0; i < kHeadOutputs / 4; ++i) {
@@ -742,8 +823,8 @@ __global__ void head_linear_kernel(const T* __restrict__ in, int in_stride, cons
             if (lane == r) mine = total;
         }
         if (lane < rows) {
-            if (gate != nullptr) mine *= sigmoid(Num<T>::load(gate + (size_t)(first + lane) * gate_stride + head));
-            Num<T>::store(out + (size_t)(first + lane) * out_stride + (size_t)head * n_out + n, mine);
+            if (gate != nullptr) mine *= sigmoid(Num<T>::load(gate + (size_t)(first + lane) * gate_stride + (layout.element_gate ? head * n_out + n : head)));
+            Num<T>::store(out + (size_t)(first + lane) * out_stride + (size_t)head * layout.out_head + n, mine);
         }
     }
 }
@@ -779,7 +860,7 @@ constexpr int kTile = 64;
 
 __global__ void __launch_bounds__(128)
 head_linear_tc_kernel(const bf16* __restrict__ in, int in_stride, const bf16* __restrict__ w, bf16* __restrict__ out, int out_stride,
-                      const bf16* __restrict__ gate, int gate_stride, int tokens, int n_in, int n_out) {
+                      const bf16* __restrict__ gate, int gate_stride, int tokens, int n_in, int n_out, HeadLayout layout) {
     grid_launch_dependents();
     grid_dependency_wait();
     extern __shared__ __align__(16) unsigned char tc_smem[];
@@ -802,15 +883,23 @@ head_linear_tc_kernel(const bf16* __restrict__ in, int in_stride, const bf16* __
     for (int i = threadIdx.x; i < kTile * pieces; i += 128) {
         const int row = i / pieces, piece = i % pieces;
         uint4 v = make_uint4(0u, 0u, 0u, 0u);
-        if (row < valid) v = *reinterpret_cast<const uint4*>(in + (size_t)(first + row) * in_stride + (size_t)head * n_in + piece * 8);
+        if (row < valid) v = *reinterpret_cast<const uint4*>(in + (size_t)(first + row) * in_stride + (size_t)head * layout.in_head + piece * 8);
         *reinterpret_cast<uint4*>(tc_smem + row * row_bytes + piece * 16) = v;
+    }
+    if (layout.turned > 0) {
+        const int half = layout.turned / 2;
+        for (int item = threadIdx.x; item < valid * half; item += 128) {
+            const size_t row = first + item / half;
+            turn_tail<bf16>(in + row * in_stride + (size_t)head * layout.in_head + n_in, out + row * out_stride + (size_t)head * layout.out_head + n_out,
+                            item % half, layout, layout.positions[row]);
+        }
     }
     const uint32_t a_rows = x_tile + (warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * row_bytes + (lane >> 4) * 16;
     float factor[2] = {1.0f, 1.0f};
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
         const int row = warp * 16 + group_id + 8 * r;
-        if (gate != nullptr && row < valid) factor[r] = sigmoid(__bfloat162float(gate[(size_t)(first + row) * gate_stride + head]));
+        if (gate != nullptr && !layout.element_gate && row < valid) factor[r] = sigmoid(__bfloat162float(gate[(size_t)(first + row) * gate_stride + head]));
     }
     for (int chunk = 0; chunk < chunks; ++chunk) {
         const int stage = chunk & 1;
@@ -838,7 +927,15 @@ head_linear_tc_kernel(const bf16* __restrict__ in, int in_stride, const bf16* __
             for (int r = 0; r < 2; ++r) {
                 const int row = warp * 16 + group_id + 8 * r;
                 if (row >= valid) continue;
-                bf16* dst = out + (size_t)(first + row) * out_stride + (size_t)head * n_out + chunk * kTile + part * 16 + tid4 * 2;
+                const int n = chunk * kTile + part * 16 + tid4 * 2;
+                bf16* dst = out + (size_t)(first + row) * out_stride + (size_t)head * layout.out_head + n;
+                if (gate != nullptr && layout.element_gate) {
+                    const bf16* g = gate + (size_t)(first + row) * gate_stride + (size_t)head * n_out + n;
+                    s[0][2 * r] *= sigmoid(__bfloat162float(g[0]));
+                    s[0][2 * r + 1] *= sigmoid(__bfloat162float(g[1]));
+                    s[1][2 * r] *= sigmoid(__bfloat162float(g[8]));
+                    s[1][2 * r + 1] *= sigmoid(__bfloat162float(g[9]));
+                }
                 *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(s[0][2 * r] * factor[r], s[0][2 * r + 1] * factor[r]);
                 *reinterpret_cast<__nv_bfloat162*>(dst + 8) = __floats2bfloat162_rn(s[1][2 * r] * factor[r], s[1][2 * r + 1] * factor[r]);
             }
@@ -966,12 +1063,12 @@ MB_EXPORT int mb_gated_attention_rows(const void* q, int q_stride, void* out, in
                                       const int* kv_lens, const float* head_bias, const void* gate, int gate_stride, int gate_kind,
                                       int sequences, int max_q_len, int heads, int kv_heads, int head_dim, int value_dim,
                                       int page_size, int softmax, float scale, float slope_exponent, const float* head_scale,
-                                      float softcap, int sink, const float* turn_cos, const float* turn_sin, int block, cudaStream_t stream) {
+                                      float softcap, int sink, const float* turn_cos, const float* turn_sin, int block, int window, cudaStream_t stream) {
     if (sequences <= 0 || max_q_len <= 0) return 0;
     if ((turn_cos == nullptr) != (turn_sin == nullptr) || (turn_cos != nullptr && value_dim % 2))
         return fail("gated_attention_rows: turning the result back needs both tables and an even value_dim (%d)", value_dim);
     if (softcap < 0.0f || (sink && !softmax)) return fail("gated_attention_rows: softcap %g, a sink without a softmax", softcap);
-    const ScoreExtras extras{head_scale, softcap, sink, turn_cos, turn_sin, block};
+    const ScoreExtras extras{head_scale, softcap, sink, turn_cos, turn_sin, block, window};
     if (head_dim <= 0 || head_dim > 2048) return fail("gated_attention_rows: head_dim %d is outside 1..2048", head_dim);
     if (value_dim <= 0 || value_dim > 512 || value_dim > v_width)
         return fail("gated_attention_rows: value_dim %d is outside 1..512 or beyond the value rows of %d", value_dim, v_width);
@@ -1041,20 +1138,20 @@ MB_EXPORT size_t mb_gated_attention_decode_scratch_floats(int sequences, int hea
     return (size_t)sequences * heads * splits * (2 + value_dim);
 }
 
-// One token per sequence (row cu_q[s] of q and out).  The keys are cut into `splits` runs of `span` pages
-// (splits * span * page_size must cover the longest sequence); `partial` holds mb_gated_attention_decode_scratch_floats floats.
+// One token per sequence (row cu_q[s] of q and out).  The keys are cut into `splits` runs of `span` pages, counted from the
+// first page a query sees (splits * span pages must cover what the longest sequence's query sees); `partial` holds mb_gated_attention_decode_scratch_floats floats.
 MB_EXPORT int mb_gated_attention_decode(const void* q, int q_stride, void* out, int out_stride, int dtype, const void* k_pool,
                                         const void* v_pool, int v_width, const int* block_table, int max_blocks, const int* cu_q,
                                         const int* kv_lens, const float* head_bias, const void* gate, int gate_stride, int gate_kind,
                                         int sequences, int heads, int kv_heads, int head_dim, int value_dim, int page_size,
                                         int softmax, float scale, float slope_exponent, int splits, int span, float* partial,
                                         const float* head_scale, float softcap, int sink, const float* turn_cos,
-                                        const float* turn_sin, int block, cudaStream_t stream) {
+                                        const float* turn_sin, int block, int window, cudaStream_t stream) {
     if (sequences <= 0) return 0;
     if ((turn_cos == nullptr) != (turn_sin == nullptr) || (turn_cos != nullptr && value_dim % 2))
         return fail("gated_attention_decode: turning the result back needs both tables and an even value_dim (%d)", value_dim);
     if (softcap < 0.0f || (sink && !softmax)) return fail("gated_attention_decode: softcap %g, a sink without a softmax", softcap);
-    const ScoreExtras extras{head_scale, softcap, sink, turn_cos, turn_sin, block};
+    const ScoreExtras extras{head_scale, softcap, sink, turn_cos, turn_sin, block, window};
     if (head_dim <= 0 || head_dim > 2048) return fail("gated_attention_decode: head_dim %d is outside 1..2048", head_dim);
     if (value_dim <= 0 || value_dim > 512 || value_dim > v_width)
         return fail("gated_attention_decode: value_dim %d is outside 1..512 or beyond the value rows of %d", value_dim, v_width);
@@ -1083,12 +1180,16 @@ MB_EXPORT int mb_gated_attention_decode(const void* q, int q_stride, void* out, 
 // tensor_cores != 0 asks for the tensor-core form where it applies (bfloat16, n_in and n_out multiples of 16, rows that
 // start on 16 bytes (in) and 4 bytes (out), at least 16 tokens).
 MB_EXPORT int mb_head_linear(const void* in, int in_stride, const void* w, void* out, int out_stride, int dtype, const void* gate,
-                             int gate_stride, int tokens, int heads, int n_in, int n_out, int tensor_cores, cudaStream_t stream) {
+                             int gate_stride, int element_gate, int tokens, int heads, int n_in, int n_out, int in_head, int out_head,
+                             int turned, const float* cos, const float* sin, const int* positions, int tensor_cores, cudaStream_t stream) {
     if (tokens <= 0 || heads <= 0) return 0;
     if (n_in <= 0 || n_out <= 0) return fail("head_linear: sizes must be positive, got %d -> %d", n_in, n_out);
+    if (turned < 0 || turned % 2 || in_head < n_in + turned || out_head < n_out + turned || (turned > 0 && (cos == nullptr || sin == nullptr || positions == nullptr)))
+        return fail("head_linear: heads of %d -> %d with a tail of %d do not fit strides %d -> %d", n_in, n_out, turned, in_head, out_head);
+    const HeadLayout layout{in_head, out_head, element_gate, turned, cos, sin, positions};
     if (heads > 65535) return fail("head_linear: %d heads exceed the grid limit 65535", heads);
     if (tensor_cores && dtype == MB_BF16 && tokens >= 16 && n_in % 16 == 0 && n_out % 16 == 0 && n_in <= 512 && in_stride % 8 == 0 &&
-        out_stride % 2 == 0 && !((uintptr_t)in & 15) && !((uintptr_t)w & 15) && !((uintptr_t)out & 3)) {
+        in_head % 8 == 0 && out_stride % 2 == 0 && out_head % 2 == 0 && !((uintptr_t)in & 15) && !((uintptr_t)w & 15) && !((uintptr_t)out & 3)) {
         const size_t smem = 3 * (size_t)tc::kTile * (n_in * 2 + 16);
         static int reserved = 0;
         if ((int)smem > reserved) {
@@ -1098,7 +1199,7 @@ MB_EXPORT int mb_head_linear(const void* in, int in_stride, const void* w, void*
         }
         MB_LAUNCH("head_linear_tc", tc::head_linear_tc_kernel, dim3((tokens + tc::kTile - 1) / tc::kTile, heads), dim3(128), smem, stream, true,
                   (const __nv_bfloat16*)in, in_stride, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)gate,
-                  gate_stride, tokens, n_in, n_out);
+                  gate_stride, tokens, n_in, n_out, layout);
         return check_launch("head_linear_tc");
     }
     const size_t smem = (size_t)kHeadRows * n_in * sizeof(float);
@@ -1107,12 +1208,12 @@ MB_EXPORT int mb_head_linear(const void* in, int in_stride, const void* w, void*
     if (dtype == MB_F32) {
         if (smem > 48 * 1024) cudaFuncSetAttribute(head_linear_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         MB_LAUNCH("head_linear", head_linear_kernel<float>, dim3(grid), dim3(128), smem, stream, true, (const float*)in, in_stride,
-                  (const float*)w, (float*)out, out_stride, (const float*)gate, gate_stride, tokens, n_in, n_out);
+                  (const float*)w, (float*)out, out_stride, (const float*)gate, gate_stride, tokens, n_in, n_out, layout);
     } else if (dtype == MB_BF16) {
         if (smem > 48 * 1024) cudaFuncSetAttribute(head_linear_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         MB_LAUNCH("head_linear", head_linear_kernel<__nv_bfloat16>, dim3(grid), dim3(128), smem, stream, true, (const __nv_bfloat16*)in,
                   in_stride, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)gate, gate_stride, tokens,
-                  n_in, n_out);
+                  n_in, n_out, layout);
     } else {
         return fail("head_linear: unknown dtype code %d", dtype);
     }
@@ -1145,4 +1246,26 @@ MB_EXPORT int mb_project_norm_rotate_store(void* q, int q_stride, const void* k,
     else
         return fail("project_norm_rotate_store: unknown dtype code %d", dtype);
     return check_launch("project_norm_rotate_store");
+}
+
+// q (or null) and k (or null: no row is stored): rows of one storage type (strides in elements); q_out [tokens, q_columns].
+MB_EXPORT int mb_latent_prepare(const void* q, int q_stride, const float* q_gain, int q_width, void* q_out, int q_columns, const void* k,
+                                int k_stride, const float* k_gain, int latent, int turned, const float* cos, const float* sin,
+                                const int* positions, float eps, void* k_pool, const int* slot_mapping, int dtype, int tokens,
+                                cudaStream_t stream) {
+    if (tokens <= 0) return 0;
+    if (turned < 0 || turned % 2 || (turned > 0 && k != nullptr && (cos == nullptr || sin == nullptr))) return fail("latent_prepare: a tail of %d numbers", turned);
+    if (q != nullptr && (q_width <= 0 || q_columns < q_width)) return fail("latent_prepare: %d query numbers in rows of %d", q_width, q_columns);
+    if (k != nullptr && latent <= 0) return fail("latent_prepare: a latent of %d numbers", latent);
+    if (dtype == MB_F32)
+        MB_LAUNCH("latent_prepare", latent_prepare_kernel<float>, dim3(tokens), dim3(128), 0, stream, true, (const float*)q, q_stride, q_gain,
+                  q_width, (float*)q_out, q_columns, (const float*)k, k_stride, k_gain, latent, turned, cos, sin, positions, eps, (float*)k_pool,
+                  slot_mapping);
+    else if (dtype == MB_BF16)
+        MB_LAUNCH("latent_prepare", latent_prepare_kernel<__nv_bfloat16>, dim3(tokens), dim3(128), 0, stream, true, (const __nv_bfloat16*)q,
+                  q_stride, q_gain, q_width, (__nv_bfloat16*)q_out, q_columns, (const __nv_bfloat16*)k, k_stride, k_gain, latent, turned, cos,
+                  sin, positions, eps, (__nv_bfloat16*)k_pool, slot_mapping);
+    else
+        return fail("latent_prepare: unknown dtype code %d", dtype);
+    return check_launch("latent_prepare");
 }

@@ -1,5 +1,5 @@
 // The tensor-core form of csrc/gated_attention.cu for steps of many tokens: bfloat16 storage, cache pages of 64
-// positions, key and value sizes fixed at compile time (-DMB_KEY_DIM, -DMB_VALUE_DIM: multiples of 16 up to 256;
+// positions, key and value sizes fixed at compile time (-DMB_KEY_DIM up to 576, -DMB_VALUE_DIM up to 256: multiples of 16;
 // -DMB_SHARED_ROWS=1: the values are the key rows themselves, so a page is copied once and read as both).
 //
 //   score(i, j) = scale * q_h(i) . k_c(j) - slope_h * (i - j) + bias_h,   weight: softmax over j <= i, or sigmoid
@@ -30,7 +30,7 @@ namespace mb {
 
 constexpr int KD = MB_KEY_DIM, VD = MB_VALUE_DIM;
 constexpr bool kSharedRows = MB_SHARED_ROWS != 0;
-static_assert(KD % 16 == 0 && KD >= 16 && KD <= 256, "key size must be a multiple of 16 in 16..256");
+static_assert(KD % 16 == 0 && KD >= 16 && KD <= 576, "key size must be a multiple of 16 in 16..576");
 static_assert(VD % 16 == 0 && VD >= 16 && VD <= 256, "value size must be a multiple of 16 in 16..256");
 static_assert(!kSharedRows || VD <= KD, "values read from key rows cannot be wider than the rows");
 constexpr int kTile = 64;  // keys per tile, one cache page
@@ -53,7 +53,14 @@ struct ScoreExtras {
     const float* turn_cos;    // [positions][VD / 2] with turn_sin: the result's pairs are turned by minus the query's position
     const float* turn_sin;
     int block;                // n > 0: a query sees only the keys of its own block of n positions (counted from 0); 0: every earlier key
+    int window;               // n > 0: a query sees only itself and the n - 1 positions before it
 };
+
+// the first position a query at `pos` sees (it never falls as the position grows)
+__device__ __forceinline__ int lowest_visible(int pos, const ScoreExtras& extras) {
+    const int of_block = extras.block > 0 ? (pos / extras.block) * extras.block : 0;
+    return extras.window > 0 ? max(of_block, pos - extras.window + 1) : of_block;
+}
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
@@ -148,8 +155,9 @@ gated_attention_tc_kernel(const bf16* __restrict__ q, int q_stride, bf16* __rest
     const int pos0 = kv_len - q_len + t0;  // position of the tile's first token
     const int last_pos = pos0 + valid - 1;
     const int t_end = last_pos / kTile + 1;
-    // with blocks of visibility the first position any row of the tile sees is the lowest row's (the bound grows with the position)
-    const int t_begin = extras.block > 0 ? ((pos0 / extras.block) * extras.block) / kTile : 0;
+    // the first position any row of the tile sees is the lowest row's
+    const int tile_low = lowest_visible(pos0, extras);
+    const int t_begin = tile_low / kTile;
     const float slope = slope_exponent != 0.0f ? exp2f(-slope_exponent * (float)(head + 1) / (float)heads) : 0.0f;
     const float bias = head_bias != nullptr ? head_bias[head] : 0.0f;
     constexpr float kLog2e = 1.4426950408889634f;
@@ -192,13 +200,13 @@ gated_attention_tc_kernel(const bf16* __restrict__ q, int q_stride, bf16* __rest
     for (int r = 0; r < 2; ++r) {
         const int row = warp * 16 + group_id + 8 * r;
         row_pos[r] = row < valid ? pos0 + row : -1;  // a row beyond the sequence sees nothing
-        row_low[r] = extras.block > 0 && row < valid ? (row_pos[r] / extras.block) * extras.block : 0;
+        row_low[r] = row < valid ? lowest_visible(row_pos[r], extras) : 0;
     }
     const int warp_last = min(pos0 + warp * 16 + 15, last_pos);  // highest position among the warp's rows
     const int warp_first_pos = pos0 + warp * 16;                  // lowest
     const bool warp_has_rows = warp * 16 < valid;
-    const int warp_first_low = extras.block > 0 ? (warp_first_pos / extras.block) * extras.block : 0;  // lowest first-visible position
-    const int warp_low = extras.block > 0 ? (warp_last / extras.block) * extras.block : 0;  // highest first-visible position among the warp's rows
+    const int warp_first_low = lowest_visible(warp_first_pos, extras);  // lowest first-visible position
+    const int warp_low = lowest_visible(warp_last, extras);  // highest first-visible position among the warp's rows
 
     for (int t = t_begin; t < t_end; ++t) {
         const int stage = t & 1;
@@ -223,19 +231,14 @@ gated_attention_tc_kernel(const bf16* __restrict__ q, int q_stride, bf16* __rest
                 *reinterpret_cast<uint4*>(rows + (first_stale + i / kPieces) * kValueRow + (i % kPieces) * 16) = make_uint4(0u, 0u, 0u, 0u);
             __syncthreads();
         }
-        if (t == t_begin && extras.block > 0) {
-            // The first tile may begin before the first key that any row of this block sees.  Those rows have weight 0 for
+        if (t == t_begin && tile_low > key_base) {
+            // The first tile begins before the first key that any row of this block sees.  Those rows have weight 0 for
             // every query, but 0 times a stray infinity or NaN is NaN, so their value rows are cleared too.
-            const int unseen = (pos0 / extras.block) * extras.block - key_base;
-            if (unseen > 0) {
-                unsigned char* rows = stage_smem + stage * kStageBytes + (kSharedRows ? 0 : kKeyTile);
-                constexpr int kPieces = kValueRow / 16;
-                if (!kSharedRows) {
-                    for (int i = threadIdx.x; i < unseen * kPieces; i += kThreads)
-                        *reinterpret_cast<uint4*>(rows + (i / kPieces) * kValueRow + (i % kPieces) * 16) = make_uint4(0u, 0u, 0u, 0u);
-                    __syncthreads();
-                }
-            }
+            unsigned char* rows = stage_smem + stage * kStageBytes + (kSharedRows ? 0 : kKeyTile);
+            constexpr int kPieces = kValueRow / 16;
+            for (int i = threadIdx.x; i < (tile_low - key_base) * kPieces; i += kThreads)
+                *reinterpret_cast<uint4*>(rows + (i / kPieces) * kValueRow + (i % kPieces) * 16) = make_uint4(0u, 0u, 0u, 0u);
+            __syncthreads();
         }
         if (warp_has_rows && key_base <= warp_last && key_base + kTile > warp_first_low) {
             const bool full = key_base + kTile - 1 <= warp_first_pos && warp * 16 + 15 < valid && key_base >= warp_low;  // no mask needed
@@ -364,11 +367,11 @@ MB_EXPORT int mb_gated_attention_tc(const void* q, int q_stride, void* out, int 
                                     const float* head_bias, const void* gate, int gate_stride, int gate_kind, int sequences,
                                     int max_q_len, int heads, int kv_heads, int page_size, int softmax, float scale,
                                     float slope_exponent, const float* head_scale, float softcap, int sink, const float* turn_cos,
-                                    const float* turn_sin, int block, cudaStream_t stream) {
+                                    const float* turn_sin, int block, int window, cudaStream_t stream) {
     if (sequences <= 0 || max_q_len <= 0) return 0;
     if ((turn_cos == nullptr) != (turn_sin == nullptr)) return fail("gated_attention_tc: turning the result back needs both tables");
     if (softcap < 0.0f || (sink && !softmax)) return fail("gated_attention_tc: softcap %g, a sink without a softmax", softcap);
-    const ScoreExtras extras{head_scale, softcap, sink, turn_cos, turn_sin, block};
+    const ScoreExtras extras{head_scale, softcap, sink, turn_cos, turn_sin, block, window};
     if (page_size != kTile) return fail("gated_attention_tc: cache pages must hold %d positions, got %d", kTile, page_size);
     if (kv_heads <= 0 || heads % kv_heads) return fail("gated_attention_tc: %d heads are no multiple of %d kv heads", heads, kv_heads);
     if (sequences > 65535 || heads > 65535) return fail("gated_attention_tc: %d sequences or %d heads exceed the grid limit 65535", sequences, heads);

@@ -705,6 +705,15 @@ expert_product_tc_kernel(const bf16* __restrict__ a, int a_stride, const bf16* _
 
 }  // namespace tc
 
+// A router without scores: chosen[t] is the row of `table` [vocab][top] that the token's id names.
+__global__ void __launch_bounds__(256)
+table_route_kernel(const int* __restrict__ table, const int* __restrict__ tokens, int* __restrict__ chosen, int entries, int top) {
+    grid_launch_dependents();
+    grid_dependency_wait();
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < entries) chosen[i] = table[(size_t)tokens[i / top] * top + i % top];
+}
+
 // out[t][c] = clamped_swish(gate[t][c], up[t][c]); grid (ceil(rows * cols / 256)); block 256.
 template <typename T>
 __global__ void clamped_swish_kernel(const T* __restrict__ gate, const T* __restrict__ up, int in_stride, T* __restrict__ out,
@@ -821,6 +830,15 @@ MB_EXPORT int mb_router_topk(const void* x, int x_stride, const void* router, in
         return fail("router_topk: unknown dtype code %d", dtype);
     }
 #undef MB_ROUTER
+    return 0;
+}
+
+// chosen [tokens][top] = the rows of `table` [vocab][top] that the tokens' ids name.
+MB_EXPORT int mb_table_route(const int* table, const int* tokens, int* chosen, int count, int top, cudaStream_t stream) {
+    if (count <= 0) return 0;
+    if (top <= 0) return fail("table_route: %d experts per token", top);
+    MB_LAUNCH("table_route", table_route_kernel, dim3((unsigned)(((size_t)count * top + 255) / 256)), dim3(256), 0, stream, true, table, tokens,
+              chosen, count * top, top);
     return 0;
 }
 

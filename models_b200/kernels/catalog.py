@@ -15,6 +15,8 @@ LIBRARIES = [
     ("mb_gated_delta", ["gated_delta.cu"], {}),
     ("mb_gated_attention", ["gated_attention.cu"], {}),
     ("mb_retention", ["retention.cu"], {}),
+    ("mb_result_norm", ["result_norm.cu"], {}),
+    ("mb_state_space", ["state_space.cu"], {}),
     ("mb_hyper_streams", ["hyper_streams.cu"], {}),
     ("mb_routed_experts", ["routed_experts.cu"], {}),
     # the tensor-core form is compiled per (key size, value size, values read from the key rows) at first use; these

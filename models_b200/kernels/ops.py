@@ -341,6 +341,103 @@ def store_rows(x: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
     return out
 
 
+def result_norm_library():
+    return load_library("mb_result_norm", ["result_norm.cu"])
+
+
+def _stream_rows(x: torch.Tensor, name: str):
+    if x.dtype != torch.float32 or x.dim() != 2 or not x.is_contiguous():
+        raise KernelError(f"{name}: the residual stream must be a contiguous float32 [rows, width] tensor")
+
+
+def _vectors(width: int, name: str, **tensors):
+    for label, t in tensors.items():
+        if t.dtype != torch.float32 or t.numel() != width or not t.is_contiguous():
+            raise KernelError(f"{name}: {label} must be contiguous float32 of {width} elements")
+
+
+def dynamic_tanh(x: torch.Tensor, alpha: float, weight: torch.Tensor, bias: torch.Tensor, out_dtype: torch.dtype,
+                 rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """tanh(alpha * x) * weight + bias of the float32 rows x [T, width] (of the rows picked by `rows`, if given), float
+    arithmetic, stored as `out_dtype`."""
+    _cuda(x, weight, bias, rows)
+    _stream_rows(x, "dynamic_tanh")
+    _vectors(x.shape[1], "dynamic_tanh", weight=weight, bias=bias)
+    _int32(rows, "rows")
+    count = rows.numel() if rows is not None else x.shape[0]
+    out = torch.empty((count, x.shape[1]), dtype=out_dtype, device=x.device)
+    lib = result_norm_library()
+    _run(lib, lib.mb_tanh_rows(_p(x), _p(rows), ctypes.c_float(alpha), _p(weight), _p(bias), _p(out), _code(out_dtype), count, x.shape[1],
+                               _stream()))
+    return out
+
+
+def _then_args(x: torch.Tensor, then, dtype, name: str):
+    """What follows an addition into the stream: None (nothing), "rows" (the new rows in `dtype`) or (alpha, weight, bias)
+    (the new rows through that dynamic tanh, in `dtype`).  Returns (arguments of the launcher, the rows to be filled or None)."""
+    if then is None:
+        return (0, ctypes.c_float(0.0), None, None, None, _F32), None
+    out = torch.empty_like(x, dtype=dtype)
+    if isinstance(then, str):
+        if then != "rows":
+            raise KernelError(f"{name}: what follows is None, 'rows' or (alpha, weight, bias), got {then!r}")
+        return (1, ctypes.c_float(0.0), None, None, _p(out), _code(dtype)), out
+    alpha, weight, bias = then
+    _cuda(weight, bias)
+    _vectors(x.shape[1], name, weight=weight, bias=bias)
+    return (2, ctypes.c_float(alpha), _p(weight), _p(bias), _p(out), _code(dtype)), out
+
+
+def result_tanh_add(x: torch.Tensor, y: torch.Tensor, alpha: float, weight: torch.Tensor, bias: torch.Tensor, then=None,
+                    dtype: Optional[torch.dtype] = None, top: int = 0, position: Optional[torch.Tensor] = None,
+                    entry_weight: float = 1.0) -> Optional[torch.Tensor]:
+    """x += tanh(alpha * y) * weight + bias in place on the float32 stream x [T, width].  `y` float32 [T, width]; with `top` n > 0
+    it holds the results of every token's n entries instead, and a token's y is entry_weight times the sum of its entries (entry
+    t * n + s in row position[t * n + s], int32, or in its own row).  `then`: see _then_args."""
+    _cuda(x, y, weight, bias, position)
+    _stream_rows(x, "result_tanh_add")
+    T, width = x.shape
+    _vectors(width, "result_tanh_add", weight=weight, bias=bias)
+    if y.dtype != torch.float32 or y.dim() != 2 or y.shape[1] != width or not y.is_contiguous() or (position is None and y.shape[0] != T * max(1, top)):
+        raise KernelError(f"result_tanh_add: results {tuple(y.shape)} {y.dtype} do not fit the stream {tuple(x.shape)} with {top} entries per row")
+    if position is not None and (not top or position.dtype != torch.int32 or position.numel() != T * top or not position.is_contiguous()):
+        raise KernelError("result_tanh_add: position must be contiguous int32 [rows * top]")
+    args, out = _then_args(x, then, dtype, "result_tanh_add")
+    lib = result_norm_library()
+    _run(lib, lib.mb_result_tanh_add(_p(x), _p(y), _p(position), int(top), ctypes.c_float(entry_weight), ctypes.c_float(alpha), _p(weight),
+                                     _p(bias), *args, T, width, _stream()))
+    return out
+
+
+def result_rms_add(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float, then=None,
+                   dtype: Optional[torch.dtype] = None) -> Optional[torch.Tensor]:
+    """x += y / sqrt(mean(y^2) + eps) * weight in place, row by row; y float32 like x.  `then`: see _then_args."""
+    _cuda(x, y, weight)
+    _stream_rows(x, "result_rms_add")
+    _vectors(x.shape[1], "result_rms_add", weight=weight)
+    if y.dtype != torch.float32 or y.shape != x.shape or not y.is_contiguous():
+        raise KernelError(f"result_rms_add: results {tuple(y.shape)} {y.dtype} do not fit the stream {tuple(x.shape)}")
+    args, out = _then_args(x, then, dtype, "result_rms_add")
+    lib = result_norm_library()
+    _run(lib, lib.mb_result_rms_add(_p(x), _p(y), _p(weight), ctypes.c_float(eps), *args, x.shape[0], x.shape[1], _stream()))
+    return out
+
+
+def side_gate(gate: torch.Tensor, table: torch.Tensor, tokens: torch.Tensor, columns: int) -> torch.Tensor:
+    """[T, columns] in the table's type: gelu_tanh(gate[t, c]) * table[tokens[t], c] for the table's columns, zeros behind them.
+    gate float32 [T, >= table columns], may be a column slice."""
+    _cuda(gate, table, tokens)
+    _columns(gate, "gate")
+    _int32(tokens, "tokens")
+    if gate.dtype != torch.float32 or not table.is_contiguous() or table.dim() != 2 or gate.shape[1] < table.shape[1] or tokens.numel() != gate.shape[0]:
+        raise KernelError(f"side_gate: gates {tuple(gate.shape)} {gate.dtype} do not fit the table {tuple(table.shape)}")
+    out = torch.empty((gate.shape[0], columns), dtype=table.dtype, device=gate.device)
+    lib = result_norm_library()
+    _run(lib, lib.mb_side_gate(_p(gate), gate.stride(0), _p(table), _p(tokens), table.shape[1], _p(out), columns, _code(table.dtype),
+                               gate.shape[0], _stream()))
+    return out
+
+
 def _columns(t: torch.Tensor, name: str):
     if t.dim() != 2 or t.stride(1) != 1:
         raise KernelError(f"{name} must be a [rows, columns] tensor (or column slice) with unit column stride")
@@ -690,11 +787,15 @@ GATED_TC_MIN_ROWS = 8  # steps that bring fewer tokens to every sequence go to t
 
 
 def gated_attention_tc_takes(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, head_dim: int, value_dim: int,
-                             max_q_len: int, gate: Optional[torch.Tensor], gate_kind: Optional[str] = "element") -> bool:
-    """bfloat16, cache pages of 64, key and value sizes multiples of 16 up to 256, 16-byte query rows."""
+                             max_q_len: int, gate: Optional[torch.Tensor], gate_kind: Optional[str] = "element",
+                             v_pool: Optional[torch.Tensor] = None) -> bool:
+    """bfloat16, cache pages of 64, key and value sizes multiples of 16 up to 256 (keys up to 576 where the values are the key
+    rows, v_pool None: one copy of a page in shared memory), 16-byte query rows."""
     if q.dtype != torch.bfloat16 or max_q_len < GATED_TC_MIN_ROWS or k_pool.shape[2] != 64:
         return False
-    if head_dim % 16 or value_dim % 16 or not 16 <= head_dim <= 256 or not 16 <= value_dim <= 256:
+    if head_dim % 16 or value_dim % 16 or not 16 <= head_dim <= 576 or not 16 <= value_dim <= 256:
+        return False
+    if v_pool is not None and head_dim > 256:
         return False
     if q.stride(0) % 8 or q.data_ptr() % 16 or out.stride(0) % 2 or out.data_ptr() % 4 or k_pool.data_ptr() % 16:
         return False
@@ -720,7 +821,7 @@ def gated_attention(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, v_
                     head_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
                     gate_kind: Optional[str] = None, kernel: Optional[str] = None, head_scale: Optional[torch.Tensor] = None,
                     softcap: float = 0.0, sink: bool = False, turn_cos: Optional[torch.Tensor] = None,
-                    turn_sin: Optional[torch.Tensor] = None, block: int = 0) -> None:
+                    turn_sin: Optional[torch.Tensor] = None, block: int = 0, window: int = 0) -> None:
     """Causal attention over the paged cache with `weights` "softmax" or "sigmoid" (independent sigmoids of the scores,
     not normalised over keys); score = scale * q.k - 2^(-slope_exponent (h + 1) / heads) * (i - j) + head_bias[h]
     (slope_exponent 0: no distance term; head_bias None: 0).  `v_pool` None: the values are the first `value_dim`
@@ -731,7 +832,7 @@ def gated_attention(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, v_
     `turn_cos`, `turn_sin` (float32 [positions, value_dim / 2]): the values were stored rotated by their own positions
     (pairs 2m, 2m + 1), and every head's sum is turned back by the query's position before any gate.
     `block` n > 0: query i sees key j <= i only if floor(i / n) = floor(j / n), blocks of n positions counted from the
-    sequence's position 0.
+    sequence's position 0; `window` n > 0: only if i - j < n.
     `kernel`: None picks the decode form for steps of one token per sequence (the keys cut into runs with a block each;
     the grid follows the page table's width, not the lengths, so that a captured step stays valid), the tensor-core form
     where it applies (bfloat16 steps of many tokens), else the form with a warp per (token, head); "decode", "tc" or
@@ -778,16 +879,20 @@ def gated_attention(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, v_
                 raise KernelError(f"gated_attention: the tables that turn the result back must be contiguous float32 [positions, {value_dim // 2}]")
     if sink and weights != "softmax":
         raise KernelError("gated_attention: a sink belongs to softmax weights")
-    if block < 0:
-        raise KernelError(f"gated_attention: a block of {block} positions")
-    extras = (_p(head_scale), ctypes.c_float(softcap), 1 if sink else 0, _p(turn_cos), _p(turn_sin), int(block))
+    if block < 0 or window < 0:
+        raise KernelError(f"gated_attention: a block of {block} positions, a window of {window}")
+    extras = (_p(head_scale), ctypes.c_float(softcap), 1 if sink else 0, _p(turn_cos), _p(turn_sin), int(block), int(window))
     softmax = 1 if weights == "softmax" else 0
     sequences = kv_lens.numel()
     gate_stride = gate.stride(0) if gate is not None else 0
     if kernel == "decode" or (kernel is None and max_q_len == 1):
         if max_q_len != 1:
             raise KernelError("the decode form takes one token per sequence")
-        runs, span = gated_decode_runs(sequences, heads, kv_heads, block_table.shape[1], _sm_count(q.device))
+        pages = block_table.shape[1]
+        for seen in (block, window):  # n positions lie in at most so many pages, wherever they start
+            if seen:
+                pages = min(pages, -(-(seen - 1) // page_size) + 1)
+        runs, span = gated_decode_runs(sequences, heads, kv_heads, pages, _sm_count(q.device))
         lib = gated_attention_library()
         lib.mb_gated_attention_decode_scratch_floats.restype = ctypes.c_size_t
         scratch = torch.empty((lib.mb_gated_attention_decode_scratch_floats(sequences, heads, value_dim, runs),), dtype=torch.float32,
@@ -799,8 +904,8 @@ def gated_attention(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, v_
             span, _p(scratch), *extras, _stream()))
         _launches[0] += 1  # two kernels
         return
-    if kernel == "tc" or (kernel is None and gated_attention_tc_takes(q, out, k_pool, head_dim, value_dim, max_q_len, gate, gate_kind)):
-        if not gated_attention_tc_takes(q, out, k_pool, head_dim, value_dim, max(max_q_len, GATED_TC_MIN_ROWS), gate, gate_kind):
+    if kernel == "tc" or (kernel is None and gated_attention_tc_takes(q, out, k_pool, head_dim, value_dim, max_q_len, gate, gate_kind, v_pool)):
+        if not gated_attention_tc_takes(q, out, k_pool, head_dim, value_dim, max(max_q_len, GATED_TC_MIN_ROWS), gate, gate_kind, v_pool):
             raise KernelError("the tensor-core form takes bfloat16, pages of 64 and key and value sizes that are multiples of 16 up to 256")
         lib = gated_attention_tc_library(head_dim, value_dim, v_pool is None)
         _run(lib, lib.mb_gated_attention_tc(
@@ -817,9 +922,13 @@ def gated_attention(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, v_
 
 
 def head_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, heads: int, gate: Optional[torch.Tensor] = None,
-                tensor_cores: bool = True) -> None:
+                tensor_cores: bool = True, gate_kind: str = "head", turned: int = 0, cos: Optional[torch.Tensor] = None,
+                sin: Optional[torch.Tensor] = None, positions: Optional[torch.Tensor] = None) -> None:
     """One small matrix per head: out[t, h, :] = weight[h] . x[t, h, :] for weight [heads, n_out, n_in], x [T, heads * n_in],
-    out [T, heads * n_out] (column slices allowed); with `gate` [T, heads], out[t, h, :] *= sigmoid(gate[t, h]).
+    out [T, heads * n_out] (column slices allowed); with `gate` [T, heads], out[t, h, :] *= sigmoid(gate[t, h]), or, gate_kind
+    "element", sigmoid of a gate [T, heads * n_out] element by element.  `turned` r > 0: every head has r more coordinates behind
+    its inputs (x [T, heads * (n_in + r)]) that pass by the matrix: rotated by the token's position (pairs (i, i + r / 2), float32
+    tables [positions, r / 2]) they are stored behind the head's outputs (out [T, heads * (n_out + r)]).
     bfloat16 steps of 16 tokens and more with sizes that are multiples of 16 run on the tensor cores unless
     `tensor_cores` is False."""
     _cuda(x, weight, out, gate)
@@ -828,17 +937,63 @@ def head_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, heads:
     if weight.dim() != 3 or weight.shape[0] != heads or not weight.is_contiguous():
         raise KernelError(f"head_linear: weight must be contiguous [{heads}, n_out, n_in], got {tuple(weight.shape)}")
     n_out, n_in = weight.shape[1], weight.shape[2]
-    if tuple(x.shape) != (out.shape[0], heads * n_in) or out.shape[1] != heads * n_out or not (x.dtype == weight.dtype == out.dtype):
+    if tuple(x.shape) != (out.shape[0], heads * (n_in + turned)) or out.shape[1] != heads * (n_out + turned) or not (x.dtype == weight.dtype == out.dtype):
         raise KernelError(f"head_linear: x {tuple(x.shape)} {x.dtype} and out {tuple(out.shape)} {out.dtype} do not fit "
                           f"{heads} matrices of {n_out} x {n_in} {weight.dtype}")
     if gate is not None:
         _columns(gate, "gate")
-        if tuple(gate.shape) != (x.shape[0], heads) or gate.dtype != x.dtype:
-            raise KernelError(f"head_linear: gate must be [{x.shape[0]}, {heads}] of x's dtype")
+        if gate_kind not in ("head", "element") or tuple(gate.shape) != (x.shape[0], heads if gate_kind == "head" else heads * n_out) or gate.dtype != x.dtype:
+            raise KernelError(f"head_linear: a gate of kind {gate_kind!r} cannot be {tuple(gate.shape)} {gate.dtype}")
+    if turned:
+        _cuda(cos, sin, positions)
+        _int32(positions, "positions")
+        for table in (cos, sin):
+            if table is None or table.dtype != torch.float32 or table.dim() != 2 or table.shape[1] * 2 != turned or not table.is_contiguous():
+                raise KernelError(f"head_linear: a tail of {turned} needs contiguous float32 tables [positions, {turned // 2}]")
     lib = gated_attention_library()
     _run(lib, lib.mb_head_linear(_p(x), x.stride(0), _p(weight), _p(out), out.stride(0), _code(x.dtype), _p(gate),
-                                 gate.stride(0) if gate is not None else 0, x.shape[0], heads, n_in, n_out,
-                                 1 if tensor_cores else 0, _stream()))
+                                 gate.stride(0) if gate is not None else 0, 1 if gate_kind == "element" else 0, x.shape[0], heads, n_in,
+                                 n_out, n_in + turned, n_out + turned, int(turned), _p(cos) if turned else None, _p(sin) if turned else None,
+                                 _p(positions) if turned else None, 1 if tensor_cores else 0, _stream()))
+
+
+def latent_prepare(q: Optional[torch.Tensor], q_gain: Optional[torch.Tensor], q_columns: int, k: Optional[torch.Tensor],
+                   k_gain: Optional[torch.Tensor], turned: int, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor],
+                   positions: torch.Tensor, eps: float, k_pool: Optional[torch.Tensor], slot_mapping: torch.Tensor) -> Optional[torch.Tensor]:
+    """What a latent attention does to its first product's rows, in one kernel.  `q` [T, n] (or None): the query's latent,
+    q / rms(q) * q_gain, returned as rows of `q_columns` >= n numbers (zeros behind the n).  `k` [T, latent + turned] (or None: the
+    layer reads another's cache): the latent / rms * k_gain and the tail rotated by the token's position (pairs
+    (i, i + turned / 2), float32 tables [positions, turned / 2]) go into the pool [pages, 1, page_size, latent + turned] at
+    `slot_mapping`.  rms(x) = sqrt(mean(x^2) + eps)."""
+    _cuda(q, q_gain, k, k_gain, cos, sin, positions, k_pool, slot_mapping)
+    _int32(positions, "positions")
+    _int32(slot_mapping, "slot_mapping")
+    rows = (q if q is not None else k).shape[0]
+    dtype = (q if q is not None else k).dtype
+    out = None
+    if q is not None:
+        _columns(q, "q")
+        if q_columns < q.shape[1] or q_gain.dtype != torch.float32 or q_gain.numel() != q.shape[1] or not q_gain.is_contiguous():
+            raise KernelError(f"latent_prepare: a query latent {tuple(q.shape)} needs a float32 gain of its size and rows that hold it")
+        out = torch.empty((rows, q_columns), dtype=dtype, device=q.device)
+    latent = 0
+    if k is not None:
+        _columns(k, "k")
+        latent = k.shape[1] - turned
+        if k.shape[0] != rows or k.dtype != dtype or k_gain.dtype != torch.float32 or k_gain.numel() != latent or not k_gain.is_contiguous():
+            raise KernelError(f"latent_prepare: rows {tuple(k.shape)} {k.dtype} with a tail of {turned} do not fit the gain or the query's rows")
+        if k_pool.dim() != 4 or k_pool.shape[1] != 1 or k_pool.shape[3] != k.shape[1] or not k_pool.is_contiguous() or k_pool.dtype != dtype:
+            raise KernelError(f"latent_prepare: the pool must be contiguous [pages, 1, page_size, {k.shape[1]}] of {dtype}")
+        if turned:
+            for table in (cos, sin):
+                if table is None or table.dtype != torch.float32 or table.dim() != 2 or table.shape[1] * 2 != turned or not table.is_contiguous():
+                    raise KernelError(f"latent_prepare: a tail of {turned} needs contiguous float32 tables [positions, {turned // 2}]")
+    lib = gated_attention_library()
+    _run(lib, lib.mb_latent_prepare(_p(q), q.stride(0) if q is not None else 0, _p(q_gain), q.shape[1] if q is not None else 0, _p(out),
+                                    int(q_columns), _p(k), k.stride(0) if k is not None else 0, _p(k_gain), latent, int(turned),
+                                    _p(cos) if turned else None, _p(sin) if turned else None, _p(positions), ctypes.c_float(eps),
+                                    _p(k_pool) if k is not None else None, _p(slot_mapping), _code(dtype), rows, _stream()))
+    return out
 
 
 RETENTION_RUN = 64  # tokens of a run when a long step's recurrence is walked in runs
@@ -1046,6 +1201,57 @@ def gated_delta_scan(conv: torch.Tensor, q_at: int, k_at: int, v_at: int, a_in: 
                                       _p(cu_q), cu_q.numel() - 1, tokens, _p(raw), _p(out), out.stride(0), ctypes.c_float(out_scale), heads,
                                       kv_heads, dim, vdim, q_at, k_at, v_at, _stream()))
     _launches[0] += 2  # three kernels: unit vectors, the walk, norm and gate
+
+
+def state_space_library():
+    return load_library("mb_state_space", ["state_space.cu"])
+
+
+def state_space_walk(rows: torch.Tensor, x_at: int, b_at: int, c_at: int, dt_in: torch.Tensor, decay: torch.Tensor, dt_bias: torch.Tensor,
+                     skip: torch.Tensor, state: torch.Tensor, state_offset: int, slots: torch.Tensor, cu_q: torch.Tensor, heads: int,
+                     groups: int, state_rows: int, vdim: int) -> torch.Tensor:
+    """The state-space recurrence over the new tokens of every sequence, token by token.  `rows` float32 [tokens, n] holds x (heads
+    heads of vdim from column x_at), B and C (groups of state_rows numbers from b_at and c_at); dt = softplus(dt_in + dt_bias) per
+    head (dt_in [tokens, heads], may be a column slice); per head, from the sequence's float32 state S [heads, state_rows, vdim]
+    at `state_offset` floats into its row of `state` (updated in place): S <- exp(decay * dt) S + dt B x^T; y = S^T C + skip x,
+    returned as float32 [tokens, heads * vdim]."""
+    _cuda(rows, dt_in, decay, dt_bias, skip, state, slots, cu_q)
+    _int32(slots, "slots")
+    _int32(cu_q, "cu_q")
+    _state_space_checks("state_space_walk", rows, x_at, b_at, c_at, dt_in, decay, dt_bias, skip, heads, groups, state_rows, vdim)
+    if rows.dtype != torch.float32:
+        raise KernelError("state_space_walk: the convolved rows must be float32")
+    at, stride = _state_rows(state, state_offset, heads * state_rows * vdim, "state_space_walk")
+    y = torch.empty((rows.shape[0], heads * vdim), dtype=torch.float32, device=rows.device)
+    lib = state_space_library()
+    _run(lib, lib.mb_state_space_walk(_p(rows), rows.stride(0), _code(rows.dtype), _p(dt_in), dt_in.stride(0), _code(dt_in.dtype), _p(decay),
+                                      _p(dt_bias), _p(skip), at, stride, _p(slots), _p(cu_q), cu_q.numel() - 1, _p(y), heads, groups,
+                                      state_rows, vdim, x_at, b_at, c_at, _stream()))
+    return y
+
+
+def _state_space_checks(name, rows, x_at, b_at, c_at, dt_in, decay, dt_bias, skip, heads, groups, state_rows, vdim):
+    _columns(rows, "rows")
+    _columns(dt_in, "dt_in")
+    if heads % groups or max(b_at, c_at) + groups * state_rows > rows.shape[1] or x_at + heads * vdim > rows.shape[1]:
+        raise KernelError(f"{name}: rows {tuple(rows.shape)} do not hold {heads} heads of {vdim} and two times {groups} groups of {state_rows}")
+    if tuple(dt_in.shape) != (rows.shape[0], heads):
+        raise KernelError(f"{name}: dt_in {tuple(dt_in.shape)} is not [{rows.shape[0]}, {heads}]")
+    _vectors(heads, name, decay=decay, dt_bias=dt_bias, skip=skip)
+
+
+def gate_part_norm(y: torch.Tensor, z: torch.Tensor, gain: torch.Tensor, eps: float, parts: int, out: torch.Tensor, out_scale: float = 1.0) -> None:
+    """out = out_scale * v / sqrt(mean(v^2) + eps) * gain with v = y * silu(z), every one of `parts` equal parts of a row by its own
+    mean.  y contiguous [tokens, width] (float32 or out's type), z and out of one type (may be column slices)."""
+    _cuda(y, z, gain, out)
+    _columns(z, "z")
+    _columns(out, "out")
+    if y.dim() != 2 or not y.is_contiguous() or y.shape != z.shape or y.shape != out.shape or z.dtype != out.dtype or y.shape[1] % parts:
+        raise KernelError(f"gate_part_norm: y {tuple(y.shape)}, z {tuple(z.shape)} and out {tuple(out.shape)} do not fit {parts} parts")
+    _vectors(y.shape[1], "gate_part_norm", gain=gain)
+    lib = state_space_library()
+    _run(lib, lib.mb_gate_part_norm(_p(y), _code(y.dtype), _p(z), z.stride(0), _p(gain), ctypes.c_float(eps), _p(out), out.stride(0),
+                                    _code(out.dtype), ctypes.c_float(out_scale), y.shape[0], y.shape[1], parts, _stream()))
 
 
 def rglru_scan(gates: torch.Tensor, per: int, u: torch.Tensor, y_in: torch.Tensor, r_bias: torch.Tensor, i_bias: torch.Tensor,
@@ -1807,6 +2013,17 @@ def router_topk(x: torch.Tensor, router: torch.Tensor, top: int, scored: bool = 
     _run(lib, lib.mb_router_topk(_p(x), x.stride(0), _p(router), _code(x.dtype), _p(chosen), _p(weights), tokens, x.shape[1], experts,
                                  top, 1 if scored else 0, _p(correction), int(groups), int(keep), ctypes.c_float(weight_scale), _stream()))
     return chosen, weights
+
+
+def table_route(table: torch.Tensor, tokens: torch.Tensor) -> torch.Tensor:
+    """chosen int32 [T, top]: the row of `table` (int32 [vocab, top]) of every token id."""
+    _cuda(table, tokens)
+    _int32(table, "table")
+    _int32(tokens, "tokens")
+    chosen = torch.empty((tokens.numel(), table.shape[1]), dtype=torch.int32, device=table.device)
+    lib = routed_experts_library()
+    _run(lib, lib.mb_table_route(_p(table), _p(tokens), _p(chosen), tokens.numel(), table.shape[1], _stream()))
+    return chosen
 
 
 class RoutePlan:

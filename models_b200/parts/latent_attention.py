@@ -5,8 +5,13 @@ q = Wq.xn (heads of `head_dim`); c = rmsnorm(Wd.xn) with a gain, `latent_dim` nu
 scale * q_i.k_j equals scale * (Uk_h^T q_i).c_j and its result sum_j w_j v_j equals Uv_h.(sum_j w_j c_j): the query is taken
 into the latent space once per token and head, the attention runs over the cached rows themselves (all heads read the same
 rows, as key and as value), and the result is taken out of the latent space once per token and head.  No key or value is
-ever expanded.  With `gated`, head h's result is multiplied by sigmoid((Wg.xn)_h); then Wo.  No positions enter.  The
+ever expanded.  With `gated`, head h's result is multiplied by sigmoid((Wg.xn)_h); then Wo.  The
 norm, the scores and the softmax are float32 in both modes.
+
+Variations (the spec says which).  Queries from a latent of their own, q = Uq.rmsnorm(Wdq.xn).  A position: every query head has
+`rotary_dim` coordinates more and the cached row as many more, one rotated key part that all heads share; the query in the latent
+space is [Uk_h^T q | rotated part], the cached row [c | rotated part], and their product is the whole score; the values are the
+row's first latent_dim numbers.  A window.  A gate per element.  Rows that another run cached (`own_rows` False).
 """
 
 from __future__ import annotations
@@ -17,38 +22,63 @@ from ..cache.kv_cache import KvRequest
 from ..kernels import ops
 from ..weights.loader import ParamRequest
 from .base import Mixer, RunContext
-from .linear import stack_rows
-from .registry import register_part
+from .linear import linear, stack_columns, stack_rows
+from .registry import build_part, register_part
 from .split import SplitPart
 
 
 class LatentAttentionMixer(SplitPart, Mixer):
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
-        self.q_width = spec.num_heads * spec.head_dim
+        if spec.gate_kind not in ("head", "element"):
+            raise ValueError(f"a gate of kind {spec.gate_kind!r} is not built (known: head, element)")
+        self.turned = spec.position.rotary_dim if spec.position is not None else 0
+        self.q_width = spec.num_heads * (spec.head_dim + self.turned)
+        self.row_width = spec.latent_dim + self.turned
         self.mid_width = spec.num_heads * spec.value_dim
+        self.rope = None
+        if spec.position is not None:
+            if spec.position.pairing != "half":
+                raise ValueError("the rotated part of a latent attention pairs coordinate i with i + rotary_dim / 2")
+            key = ("position", spec.position, runtime.max_positions)
+            if key not in runtime.shared:
+                runtime.shared[key] = build_part("position", spec.position, runtime)
+            self.rope = runtime.shared[key]
 
     def _first(self):
-        return ("q", "down", "gate") if self.spec.gated else ("q", "down")
+        """The matrices that read the normalised rows: (role, rows)."""
+        s = self.spec
+        out = [("down_q", s.query_latent) if s.query_latent else ("q", self.q_width)]
+        if s.own_rows:
+            out.append(("down", self.row_width))
+        if s.gated:
+            out.append(("gate", s.num_heads if s.gate_kind == "head" else self.mid_width))
+        return out
 
     def parameters(self):
         s, n = self.spec, self.spec.weights
-        widths = {"q": self.q_width, "down": s.latent_dim, "gate": s.num_heads}
-        out = [ParamRequest(n[r], (widths[r], s.hidden_size)) for r in self._first()]
-        out += [ParamRequest(n["down_norm"], (s.latent_dim,), "gain"),
-                ParamRequest(n["up_k"], (self.q_width, s.latent_dim)),
+        out = [ParamRequest(n[role], (rows, s.hidden_size)) for role, rows in self._first()]
+        if s.query_latent:
+            out += [ParamRequest(n["down_q_norm"], (s.query_latent,), "gain"), ParamRequest(n["up_q"], (self.q_width, s.query_latent))]
+        if s.own_rows:
+            out.append(ParamRequest(n["down_norm"], (s.latent_dim,), "gain"))
+        out += [ParamRequest(n["up_k"], (s.num_heads * s.head_dim, s.latent_dim)),
                 ParamRequest(n["up_v"], (self.mid_width, s.latent_dim)),
                 ParamRequest(n["o"], (s.hidden_size, self.mid_width))]
         return out
 
     def load(self, tensors):
         s, n, rt = self.spec, self.spec.weights, self.runtime
-        first = [rt.matrix(tensors[n[r]]) for r in self._first()]
+        first = [rt.matrix(tensors[n[role]]) for role, _ in self._first()]
         if len({m.dtype for m in first}) > 1:
             first = [m.float() for m in first]
-        self.w_in, self.starts = stack_rows(first)
+        self.w_in, starts = stack_rows(first)
+        self.columns = {role: slice(at, at + rows) for (role, rows), at in zip(self._first(), starts)}
         self.w_o = rt.matrix(tensors[n["o"]])
-        self.latent_gain = rt.vector(tensors[n["down_norm"]])
+        self.latent_gain = rt.vector(tensors[n["down_norm"]]) if s.own_rows else None
+        if s.query_latent:
+            self.query_gain = rt.vector(tensors[n["down_q_norm"]])
+            self.up_q, _, _ = stack_columns([rt.matrix(tensors[n["up_q"]])])  # (columns of padding meet zeros)
         dtype = rt.compute_dtype
         # per head: [latent_dim, head_dim] takes a query into the latent space, [value_dim, latent_dim] a result out of it
         self.into_latent = rt.matrix(tensors[n["up_k"]]).to(dtype).view(s.num_heads, s.head_dim, s.latent_dim).transpose(1, 2).contiguous()
@@ -61,30 +91,33 @@ class LatentAttentionMixer(SplitPart, Mixer):
         return self.w_o
 
     def kv_request(self):
-        return KvRequest(1, self.spec.latent_dim, None, 0)  # one row per position, read as key and as value
+        # one row per position, read as key and as value
+        return KvRequest(1, self.row_width, self.spec.window, 0)
 
     def inner(self, proj: torch.Tensor, mid: torch.Tensor, batch, run: RunContext, scale: float = 1.0) -> None:
         s = self.spec
         if run.k_pool is None:
             raise RuntimeError("the latent attention mixer needs a cache pool; its run has none")
-        if not run.writes_cache:
-            raise RuntimeError("this mixer writes the cache it reads; a run that reads another run's cache is not built for it")
+        if run.writes_cache != s.own_rows:
+            raise RuntimeError("this mixer makes rows of its own and its run reads another's, or the other way round")
         if scale != 1.0:
             raise ValueError("this mixer's result cannot be scaled on its way out")
         group = batch.groups[run.group]
-        at = self.starts
-        q = proj[:, at[0]:at[0] + self.q_width]
-        down = proj[:, at[1]:at[1] + s.latent_dim]
-        gate = proj[:, at[2]:at[2] + s.num_heads] if s.gated else None
-        ops.norm_store(None, down, None, batch.positions, None, self.latent_gain, s.eps, 0.0, 1, run.k_pool, None,
-                       group.slot_mapping, 0, 1, s.latent_dim, 0)
+        part = lambda role: proj[:, self.columns[role]] if role in self.columns else None  # noqa: E731
+        cos, sin = (self.rope.cos, self.rope.sin) if self.rope is not None else (None, None)
+        down_q, down, gate = part("down_q"), part("down"), part("gate")
+        q_rows = None
+        if down_q is not None or down is not None:
+            q_rows = ops.latent_prepare(down_q, self.query_gain if down_q is not None else None, self.up_q.shape[1] if down_q is not None else 0,
+                                        down, self.latent_gain, self.turned, cos, sin, batch.positions, s.eps, run.k_pool, group.slot_mapping)
+        q = part("q") if down_q is None else linear(q_rows, self.up_q, proj.dtype)
         rows = proj.shape[0]
-        q_latent = torch.empty((rows, s.num_heads * s.latent_dim), dtype=proj.dtype, device=proj.device)
-        ops.head_linear(q, self.into_latent, q_latent, s.num_heads)
-        mixed = torch.empty_like(q_latent)
+        q_latent = torch.empty((rows, s.num_heads * self.row_width), dtype=proj.dtype, device=proj.device)
+        ops.head_linear(q, self.into_latent, q_latent, s.num_heads, turned=self.turned, cos=cos, sin=sin, positions=batch.positions)
+        mixed = torch.empty((rows, s.num_heads * s.latent_dim), dtype=proj.dtype, device=proj.device)
         ops.gated_attention(q_latent, mixed, run.k_pool, None, group.block_table, batch.cu_q, batch.kv_lens, batch.max_q_len,
-                            s.num_heads, 1, s.latent_dim, s.latent_dim, "softmax", s.scale)
-        ops.head_linear(mixed, self.out_of_latent, mid, s.num_heads, gate)
+                            s.num_heads, 1, self.row_width, s.latent_dim, "softmax", s.scale, window=s.window or 0)
+        ops.head_linear(mixed, self.out_of_latent, mid, s.num_heads, gate, gate_kind=s.gate_kind)
 
 
 register_part("mixer", "latent_attention", LatentAttentionMixer)

@@ -30,5 +30,9 @@ class RmsNorm(Part):
                 write_x: bool = True) -> torch.Tensor:
         return ops.add_rmsnorm(x, delta, self.weight, self.spec.eps, self.runtime.compute_dtype, rows, write_x)
 
+    def add_result(self, x: torch.Tensor, y: torch.Tensor, then) -> Optional[torch.Tensor]:
+        """x += norm(y) for a sublayer's float32 result y; `then`: what becomes of the new rows (ops.result_rms_add)."""
+        return ops.result_rms_add(x, y, self.weight, self.spec.eps, then, self.runtime.compute_dtype)
+
 
 register_part("norm", "rmsnorm", RmsNorm)

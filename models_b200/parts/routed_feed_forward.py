@@ -10,7 +10,8 @@ s + correction (a tensor), restricted to the outputs of the `keep_groups` best o
 (a group counts by its largest choice score), and the weights are weight_scale * s of the chosen, not renormalised.  Identity
 experts: the router's last outputs stand for experts without tensors whose result is their input; their entries skip both
 products and enter the weighted sum as the token's own row.  An expert without clamps and without the one added to the up
-branch (limit +inf, slope 1, up_offset 0: silu(g) * u).  A shared expert that is added as it is, without a gate.
+branch (limit +inf, slope 1, up_offset 0: silu(g) * u).  A shared expert that is added as it is, without a gate.  A "table"
+rule without any router: an integer table gives every token id its experts, each with the weight 1 / top.
 
 The step's (token, choice) entries are sorted by expert on the device; the experts' two products are then grouped products
 over the sorted rows (a block a tile of one expert's rows), whose grids depend on the number of tokens only -- nothing comes
@@ -22,6 +23,9 @@ is float32 [tokens, width]: the weighted sum of the chosen experts' float32 resu
 
 from __future__ import annotations
 
+from dataclasses import dataclass
+from typing import Optional
+
 import torch
 
 from ..kernels import ops
@@ -31,14 +35,29 @@ from .linear import linear, stack_rows
 from .registry import register_part
 
 
+@dataclass
+class ExpertResults:
+    """The chosen experts' float32 results, still to be summed with equal weights: token t's sum is `weight` times the rows
+    position[t * top + s] (position None: t * top + s itself) of `rows`."""
+
+    rows: torch.Tensor
+    position: Optional[torch.Tensor]
+    top: int
+    weight: float
+
+
 class RoutedFeedForward(Part):
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
         self.outputs = spec.num_experts + spec.identity_experts  # what the router has: experts, then identity experts
         if not 1 <= spec.top <= self.outputs:
             raise ValueError(f"top {spec.top} of {self.outputs} router outputs")
-        if spec.rule not in ("top_logits", "scored"):
-            raise ValueError(f"router rule {spec.rule!r} is not built (known: top_logits, scored)")
+        if spec.rule not in ("top_logits", "scored", "table"):
+            raise ValueError(f"router rule {spec.rule!r} is not built (known: top_logits, scored, table)")
+        if spec.rule == "table":
+            if spec.identity_experts or spec.shared is not None:
+                raise ValueError("identity experts and a shared expert are not built beside a table of experts")
+            self.forward_results = self._forward_results  # (equal weights: whoever adds the result may sum it too)
         if spec.rule != "scored" and (spec.correction or spec.groups != 1 or spec.weight_scale != 1.0):
             raise ValueError("a correction, groups and a weight scale belong to the scored rule")
         if self.outputs % spec.groups or not 1 <= spec.keep_groups <= spec.groups:
@@ -50,7 +69,10 @@ class RoutedFeedForward(Part):
     def parameters(self):
         s, n = self.spec, self.spec.weights
         ff, W = s.expert.intermediate_size, s.hidden_size
-        out = [ParamRequest(n["router"], (self.outputs, W))]
+        if s.rule == "table":
+            out = [ParamRequest(n["table"], (s.vocab_size, s.top), "table", limit=s.num_experts)]
+        else:
+            out = [ParamRequest(n["router"], (self.outputs, W))]
         if s.correction:
             out.append(ParamRequest(n["correction"], (self.outputs,), "bias"))
         for role, shape in (("gate", (ff, W)), ("up", (ff, W)), ("down", (W, ff))):
@@ -65,7 +87,11 @@ class RoutedFeedForward(Part):
 
     def load(self, tensors):
         s, n, rt = self.spec, self.spec.weights, self.runtime
-        self.router = rt.matrix(tensors[n["router"]])
+        self.router = self.table = None
+        if s.rule == "table":
+            self.table = tensors[n["table"]].to(rt.device, torch.int32).contiguous()
+        else:
+            self.router = rt.matrix(tensors[n["router"]])
         self.correction = rt.vector(tensors[n["correction"]]) if s.correction else None
         stacked = {}
         for role in ("gate", "up", "down"):
@@ -73,9 +99,9 @@ class RoutedFeedForward(Part):
             if len({m.dtype for m in parts}) > 1:
                 parts = [m.float() for m in parts]
             stacked[role] = torch.stack(parts, dim=0).contiguous()
-        if len({m.dtype for m in stacked.values()} | {self.router.dtype}) > 1:
+        if len({m.dtype for m in stacked.values()} | ({self.router.dtype} if self.router is not None else set())) > 1:
             stacked = {r: m.float() for r, m in stacked.items()}
-            self.router = self.router.float()
+            self.router = self.router.float() if self.router is not None else None
         # gate and up matrices in one buffer (all experts' gate rows, then all up rows): the grouped tensor-core product
         # reads both through one map
         self.w_gate_up = torch.stack([stacked["gate"], stacked["up"]], dim=0).contiguous()
@@ -89,13 +115,10 @@ class RoutedFeedForward(Part):
             self.shared_in, self.shared_starts = stack_rows(first)
             self.shared_down = rt.matrix(tensors[n["shared_down"]])
 
-    def forward_wide(self, xn: torch.Tensor, batch=None, run=None) -> torch.Tensor:
-        """float32 [tokens, width]."""
+    def _experts(self, x: torch.Tensor, chosen: torch.Tensor):
+        """The chosen experts' float32 results and the row of every (token, choice) entry among them (None: in entry order)."""
         s = self.spec
         e = s.expert
-        x = xn if xn.dtype == self.router.dtype else xn.to(self.router.dtype)
-        chosen, weights = ops.router_topk(x, self.router, s.top, scored=s.rule == "scored", correction=self.correction,
-                                          groups=s.groups, keep=s.keep_groups, weight_scale=s.weight_scale)
         position = None
         # (an identity expert's id lies beyond the experts': the sorting and the products leave its entries out, and the
         # weighted sum takes the token's own row for them)
@@ -112,6 +135,24 @@ class RoutedFeedForward(Part):
             plan = ops.route_sort(chosen, s.num_experts)
             mid = ops.expert_first_product(x, self.w_gate, self.w_up, plan, e.limit, e.swish_slope, up_offset=e.up_offset)
             slot_out = ops.expert_second_product(mid, self.w_down, plan)
+        return slot_out, position
+
+    def _forward_results(self, xn: torch.Tensor, batch, run=None) -> ExpertResults:
+        x = xn if xn.dtype == self.w_down.dtype else xn.to(self.w_down.dtype)
+        rows, position = self._experts(x, ops.table_route(self.table, batch.tokens))
+        return ExpertResults(rows, position, self.spec.top, 1.0 / self.spec.top)
+
+    def forward_wide(self, xn: torch.Tensor, batch=None, run=None) -> torch.Tensor:
+        """float32 [tokens, width]."""
+        s = self.spec
+        if s.rule == "table":
+            r = self._forward_results(xn, batch, run)
+            weights = torch.full((xn.shape[0], r.top), r.weight, dtype=torch.float32, device=xn.device)
+            return ops.expert_combine(r.rows, weights, position=r.position)
+        x = xn if xn.dtype == self.router.dtype else xn.to(self.router.dtype)
+        chosen, weights = ops.router_topk(x, self.router, s.top, scored=s.rule == "scored", correction=self.correction,
+                                          groups=s.groups, keep=s.keep_groups, weight_scale=s.weight_scale)
+        slot_out, position = self._experts(x, chosen)
         identity = dict(chosen=chosen, experts=s.num_experts, rows=x) if s.identity_experts else {}
         if self.shared_in is None:
             return ops.expert_combine(slot_out, weights, position=position, **identity)

@@ -32,11 +32,13 @@ class WeightsError(ValueError):
 @dataclass(frozen=True)
 class ParamRequest:
     """A tensor a part needs.  kind: "matrix" (used by matrix products, random init N(0, std)),
-    "gain" (a norm's weight, random init 1 + N(0, gain_std)), "bias" (random init N(0, std))."""
+    "gain" (a norm's weight, random init 1 + N(0, gain_std)), "bias" (random init N(0, std)), "table" (integers in
+    [0, limit), those of a row all different, random init uniform)."""
 
     name: str
     shape: Tuple[int, ...]
     kind: str = "matrix"
+    limit: int = 0
 
 
 def _open_files(folder: Path) -> Tuple[List[SafetensorsFile], Dict[str, SafetensorsFile]]:
@@ -88,6 +90,16 @@ def check_names_and_shapes(requests: Mapping[str, ParamRequest], found: Mapping[
     raise WeightsError("\n".join(lines), missing, unexpected, wrong)
 
 
+def _check_table(folder, request: ParamRequest, t: torch.Tensor) -> None:
+    if t.dtype != torch.int32:
+        raise WeightsError(f"{folder}: {request.name} must be a table of integers, it is stored as {t.dtype}")
+    if t.numel() and not (0 <= int(t.min()) and int(t.max()) < request.limit):
+        raise WeightsError(f"{folder}: {request.name} holds integers outside [0, {request.limit})")
+    ordered = t.sort(dim=-1).values
+    if bool((ordered[..., 1:] == ordered[..., :-1]).any()):
+        raise WeightsError(f"{folder}: {request.name} has a row that names the same entry twice")
+
+
 def load_tensors(folder, requests: Mapping[str, ParamRequest], ignored: Sequence[str] = (),
                  duplicates: Mapping[str, str] = {}) -> Dict[str, torch.Tensor]:
     """Host tensors for every requested name.  bfloat16 stays bfloat16, a tensor stored in 32-bit
@@ -105,6 +117,9 @@ def load_tensors(folder, requests: Mapping[str, ParamRequest], ignored: Sequence
             del found[name]
         check_names_and_shapes(requests, found, str(folder))
         tensors = {name: by_name[name].tensor(name) for name in requests}
+        for name, request in requests.items():
+            if request.kind == "table":
+                _check_table(folder, request, tensors[name])
         for name in repeated:
             original = duplicates[name]
             copy = by_name[name].tensor(name)

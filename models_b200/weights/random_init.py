@@ -22,7 +22,7 @@ from .safetensors_io import write_safetensors
 
 def random_tensors(requests: Mapping[str, ParamRequest], seed: int, std: float = 0.02, gain_std: float = 0.1,
                    dtype: torch.dtype = torch.bfloat16, device="cpu") -> Dict[str, torch.Tensor]:
-    """Matrices and biases N(0, std); norm gains 1 + N(0, gain_std).  Drawn in float32, then rounded
+    """Matrices and biases N(0, std); norm gains 1 + N(0, gain_std); tables int32, uniform.  Others drawn in float32, then rounded
     to `dtype`.  Values come from a counter-based generator keyed by (seed, tensor name)
     (weights/philox_normal.py): on a CUDA device a kernel draws them in place, on the host numpy does,
     and both give the same bits."""
@@ -35,6 +35,9 @@ def random_tensors(requests: Mapping[str, ParamRequest], seed: int, std: float =
         count = 1
         for n in shape:
             count *= n
+        if request.kind == "table":
+            out[name] = _random_table(shape, request.limit, key).to(device)
+            continue
         if device.type == "cuda":
             from ..kernels import ops
 
@@ -43,6 +46,13 @@ def random_tensors(requests: Mapping[str, ParamRequest], seed: int, std: float =
             values = torch.from_numpy(normal_float32(count, key, mean, scale)).reshape(shape)
             out[name] = values.to(dtype)
     return out
+
+
+def _random_table(shape, limit: int, key) -> torch.Tensor:
+    """Integers in [0, limit): a row starts at a drawn number and counts on (modulo limit), so its entries differ."""
+    rows, top = shape
+    start = torch.from_numpy(normal_float32(rows, key, 0.0, 4096.0)).abs().to(torch.int64)
+    return ((start[:, None] + torch.arange(top)) % limit).to(torch.int32)
 
 
 def write_random_model(folder, config, seed: int, std: float = 0.02, gain_std: float = 0.1,
