@@ -1002,6 +1002,203 @@ def rolevik_kernels(z, peak, prompt=2048, batch=8, context=1536):
     return out
 
 
+# --design mabivik: the Mabivik decoder (layers with a dynamic tanh before and after each sublayer and the token let in once more; a
+# gated delta rule, a latent attention with a rotated shared key and a window, a state-space recurrence; experts by a table of token
+# ids) beside a Rolevik of equal size: the model of this package whose layers are nearest (the same delta rule, routed experts, norms
+# on the results); equal size counts the parameters a token uses.
+
+MABIVIK_SIZES = {
+    # width, layers (MABIVIK_ORDER in turn), the delta rule's heads, query/key heads, key and value size, the attention's heads, key
+    # size, rotated size, value size, query rank, latent rank and window, the state space's heads, columns, rows, groups, experts,
+    # chosen per token, an expert's ff, the side input's size
+    "s": dict(width=1024, layers=8, delta_heads=8, delta_kv_heads=4, dim=64, vdim=128, heads=8, rot_dim=64, q_rank=512, kv_rank=256, window=512,
+              space_heads=32, space_vdim=64, space_state=128, groups=2, experts=16, top=2, expert_ff=1024, side=64),
+    "m": dict(width=2048, layers=16, delta_heads=16, delta_kv_heads=8, dim=64, vdim=128, heads=16, rot_dim=64, q_rank=1024, kv_rank=256, window=1024,
+              space_heads=64, space_vdim=64, space_state=128, groups=2, experts=32, top=4, expert_ff=1024, side=128),
+}
+MABIVIK_ORDER = ("delta", "latent", "space", "reader")  # reader: an attention over the rows of the turn's other attention
+
+
+def mabivik_config(z):
+    D, DV = z["dim"], z["vdim"]
+    latent = {"heads": z["heads"], "dim": D, "rot_dim": z["rot_dim"], "vdim": DV, "q_rank": z["q_rank"], "kv_rank": z["kv_rank"],
+              "scale": (D + z["rot_dim"]) ** -0.5, "mask": {"size": z["window"]},
+              "rot": {"dims": z["rot_dim"], "base": 500000.0, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    mlp = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"]}, "expert": {"ff": z["expert_ff"]}}
+    layers = []
+    for i in range(z["layers"]):
+        kind = MABIVIK_ORDER[i % 4]
+        if kind == "delta":
+            entry = ("delta", {"heads": z["delta_heads"], "kv_heads": z["delta_kv_heads"], "dim": D, "vdim": DV, "conv": 4})
+        elif kind == "space":
+            entry = ("mamba2", {"heads": z["space_heads"], "vdim": z["space_vdim"], "state": z["space_state"], "groups": z["groups"],
+                                "norm_groups": z["groups"], "conv": 4})
+        else:
+            entry = ("latent_attention", dict(latent, kv_from=i - 2) if kind == "reader" else latent)
+        layers.append({"type": entry[0], "mixer": entry[1], "mlp": mlp})
+    return {"architecture": "Mabivik", "vocab": DESIGN_VOCAB, "width": z["width"], "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "logit_scale": 1.0, "token_side": {"dim": z["side"]}, "layers": layers}
+
+
+def mabivik_layer_params(z):
+    """Matrix parameters a token uses in a layer (of the experts only the chosen ones), averaged over the four layers of a turn."""
+    w, d, dv, dh, dg, h = (z[k] for k in ("width", "dim", "vdim", "delta_heads", "delta_kv_heads", "heads"))
+    inner = z["space_heads"] * z["space_vdim"]
+    attention = w * z["q_rank"] + z["q_rank"] * h * (d + z["rot_dim"]) + h * (d + dv) * z["kv_rank"] + 2 * w * h * dv
+    mixers = {"delta": w * (2 * dg * d + 2 * dh * dv + 2 * dh) + dh * dv * w,
+              "latent": attention + w * (z["kv_rank"] + z["rot_dim"]), "reader": attention,
+              "space": w * (2 * inner + 2 * z["groups"] * z["space_state"] + z["space_heads"]) + inner * w}
+    return sum(mixers.values()) // 4 + z["top"] * 3 * w * z["expert_ff"] + 2 * w * z["side"]
+
+
+def rolevik_of_equal_size(z):
+    """A Rolevik of the bench's size with the same width and layers whose dense feed-forward width (a multiple of 256) makes a layer's
+    parameters equal to those a Mabivik token uses."""
+    zr = next(dict(r) for r in ROLEVIK_SIZES.values() if r["width"] == z["width"])
+    zr["ff"] = 0
+    zr["ff"] = max(256, round((mabivik_layer_params(z) - rolevik_layer_params(zr)) / (1.5 * z["width"]) / 256) * 256)  # (half the layers are dense)
+    return rolevik_config(zr)
+
+
+def mabivik_kernels(z, peak, prompt=2048, batch=8, context=1536):
+    """The design's kernels alone beside the like kernels of the other models at equal sizes, each with its fraction of the
+    measured peak that bounds it."""
+    import torch
+
+    from models_b200.kernels import ops
+
+    dev, bf = "cuda", torch.bfloat16
+    H, D, R, DV, W, K, Q = (z[k] for k in ("heads", "dim", "rot_dim", "vdim", "width", "kv_rank", "q_rank"))
+    SH, SP, SN, SG = (z[k] for k in ("space_heads", "space_vdim", "space_state", "groups"))
+    E, top, F = z["experts"], z["top"], z["expert_ff"]
+    page, taps, window = 64, 4, z["window"]
+    out = {}
+
+    def rated(us, flops=None, moved=None):
+        if flops is not None:
+            return {"us": us, "tflops": flops / us / 1e6, "frac_of_bf16_peak": flops / us / 1e6 / peak["bf16_tflops"]}
+        return {"us": us, "gbs": moved / us / 1e3, "frac_of_hbm_peak": moved / us / 1e3 / peak["hbm_gbs"]}
+
+    longest = max(prompt, context)
+    angle = torch.arange(longest, dtype=torch.float32, device=dev)[:, None]
+    cos, sin = (f(angle * torch.rand((1, R // 2), device=dev)).contiguous() for f in (torch.cos, torch.sin))
+    for name, rows, cu_q, lengths, q_len in (("prompt", prompt, [0, prompt], [prompt], prompt),
+                                             ("decode", batch, list(range(batch + 1)), [context] * batch, 1)):
+        sequences = len(lengths)
+        cu = torch.tensor(cu_q, dtype=torch.int32, device=dev)
+        kv = torch.tensor(lengths, dtype=torch.int32, device=dev)
+        slots = torch.arange(sequences, dtype=torch.int32, device=dev)
+        seen = sum(min(p + 1, window) for n in lengths for p in range(n - q_len, n))  # (query, key) pairs of a head inside the window
+        pairs = sum(sum(range(n - q_len + 1, n + 1)) for n in lengths)                # and without one
+        positions = torch.cat([torch.arange(n - q_len, n) for n in lengths]).to(torch.int32).to(dev)
+        pages = sequences * (-(-lengths[0] // page))
+        table = (torch.arange(pages, dtype=torch.int32, device=dev) + 1).reshape(sequences, -1).contiguous()
+        mapping = (torch.arange(rows, dtype=torch.int32, device=dev) + page)
+        # latent attention: queries in the latent space with a rotated part, a window; beside Lovurax's (no rotated part, no window)
+        for title, tail, win, used in (("latent_attention", R, window, seen), ("latent_attention_lovurax", 0, 0, pairs)):
+            pool = torch.randn((pages + 1, 1, page, K + tail), device=dev).to(bf)
+            q, o = torch.randn((rows, H * (K + tail)), device=dev).to(bf), torch.empty((rows, H * K), dtype=bf, device=dev)
+            us = time_kernel(lambda: ops.gated_attention(q, o, pool, None, table, cu, kv, q_len, H, 1, K + tail, K, "softmax", D ** -0.5, window=win))
+            out[f"{name}_{title}"] = rated(us, flops=used * H * (2 * (K + tail) + 2 * K)) if q_len > 1 else \
+                rated(us, moved=sum(min(n, win or n) for n in lengths) * (K + tail) * 2)
+            # the products per head around it (the query's rotated part passes by; gates per element or per head)
+            x = torch.randn((rows, H * (D + tail)), device=dev).to(bf)
+            into, outof = torch.randn((H, K, D), device=dev).to(bf), torch.randn((H, DV, K), device=dev).to(bf)
+            gate = torch.randn((rows, H * DV if tail else H), device=dev).to(bf)
+            y = torch.empty((rows, H * DV), dtype=bf, device=dev)
+            us = time_kernel(lambda: (ops.head_linear(x, into, q, H, turned=tail, cos=cos, sin=sin, positions=positions),
+                                      ops.head_linear(o, outof, y, H, gate, gate_kind="element" if tail else "head")))
+            out[f"{name}_head_products" + ("" if tail else "_lovurax")] = rated(us, flops=rows * H * 2 * K * (D + DV)) if q_len > 1 else \
+                rated(us, moved=H * K * (D + DV) * 2 + rows * H * (D + K + K + DV) * 2)
+            # what stands before it: the query latent's norm, the cached row's norm and rotation; beside Lovurax's norm and store
+            first = torch.randn((rows, Q + K + tail), device=dev).to(bf)
+            gq, gk = torch.ones(Q, device=dev), torch.ones(K, device=dev)
+            if tail:
+                us = time_kernel(lambda: ops.latent_prepare(first[:, :Q], gq, Q, first[:, Q:], gk, tail, cos, sin, positions, 1e-6, pool, mapping))
+                out[f"{name}_latent_prepare"] = rated(us, moved=rows * 4 * (Q + K + tail))
+            else:
+                us = time_kernel(lambda: ops.norm_store(None, first[:, Q:], None, positions, None, gk, 1e-6, 0.0, 1, pool, None, mapping, 0, 1, K, 0))
+                out[f"{name}_norm_store_lovurax"] = rated(us, moved=rows * 4 * K)
+        # the state-space recurrence (convolution, chunks or walk, gate and norm) beside Lovurax's retention of the same state size
+        C = SH * SP + 2 * SG * SN
+        floats = SH * SN * SP
+        state = torch.zeros((sequences + 1, floats + (taps - 1) * C), dtype=torch.float32, device=dev)
+        proj = torch.randn((rows, SH * SP + C + SH), device=dev).to(bf)
+        conv_w, conv_b = torch.randn((C, taps), device=dev) * 0.4, torch.randn(C, device=dev)
+        decay, dt_bias, skip, gain = -torch.rand(SH, device=dev), torch.randn(SH, device=dev), torch.ones(SH, device=dev), torch.ones(SH * SP, device=dev)
+        mid = torch.empty((rows, SH * SP), dtype=bf, device=dev)
+        z_in, xbc, dt = proj[:, :SH * SP], proj[:, SH * SP:SH * SP + C], proj[:, SH * SP + C:]
+        at = (0, SH * SP, SH * SP + SG * SN)
+        chunked = ops.state_space_chunks_takes(bf, SN, SP, q_len, at[1])
+        conv = lambda: ops.short_conv(xbc, conv_w, state, floats, slots, cu, q_len, out_bias=conv_b, activation="silu", store_tail=True,  # noqa: E731
+                                      out_dtype=bf if chunked else torch.float32)
+
+        def recur(c):
+            if chunked:
+                return ops.state_space_chunks(c, *at, dt, decay, dt_bias, skip, state, 0, slots, cu, q_len, SH, SG, SN, SP)
+            return ops.state_space_walk(c, *at, dt, decay, dt_bias, skip, state, 0, slots, cu, SH, SG, SN, SP)
+
+        moved = rows * (2 * SH * SP + C + SH) * 2 + sequences * floats * 8
+        us = time_kernel(lambda: ops.gate_part_norm(recur(conv()), z_in, gain, 1e-6, SG, mid))
+        out[f"{name}_state_space"] = dict(rated(us, moved=moved), fp32_tflops=rows * SH * 4 * SN * SP / us / 1e6)
+        c = conv()
+        out[f"{name}_state_space_recurrence_alone"] = {"us": time_kernel(lambda: recur(c))}
+        y = recur(c)
+        out[f"{name}_state_space_norm_alone"] = {"us": time_kernel(lambda: ops.gate_part_norm(y, z_in, gain, 1e-6, SG, mid))}
+        out[f"{name}_state_space_conv_alone"] = {"us": time_kernel(conv)}
+        RH, RD, RV = SH * SP * SN // (64 * 128), 64, 128
+        rstate = torch.zeros((sequences + 1, RH, RD, RV), dtype=torch.float32, device=dev)
+        rproj = torch.randn((rows, 2 * RH * RD + 2 * RH * RV), device=dev).to(bf)
+        a, b, e = RH * RD, 2 * RH * RD, 2 * RH * RD + RH * RV
+        ro, rdecay = torch.empty((rows, RH * RV), dtype=bf, device=dev), torch.full((RH,), 0.99, device=dev)
+        us = time_kernel(lambda: ops.retention_scan(rproj[:, :a], rproj[:, a:b], rproj[:, b:e], rproj[:, e:], positions, None, None, 0, rdecay, 1.0,
+                                                    1e-6, rstate, slots, cu, RH, RD, RV, ro, 1.0, q_len))
+        out[f"{name}_retention_lovurax"] = dict(rated(us, moved=rows * (2 * RH * RD + 3 * RH * RV) * 2 + sequences * floats * 8),
+                                                fp32_tflops=rows * RH * 4 * RD * RV / us / 1e6)
+        # experts by a table of token ids beside Rolevik's scored router, both with the plain gated experts
+        x = torch.randn((rows, W), device=dev).to(bf)
+        tokens = torch.randint(0, DESIGN_VOCAB, (rows,), dtype=torch.int32, device=dev)
+        chosen_by = torch.stack([torch.randperm(E, device=dev)[:top] for _ in range(1024)]).to(torch.int32).repeat(DESIGN_VOCAB // 1024, 1).contiguous()
+        router = (torch.randn((E, W), device=dev) * 0.02).to(bf)
+        w_gate_up = (torch.randn((2, E, F, W), device=dev) * 0.02).to(bf)
+        w_down = (torch.randn((E, W, F), device=dev) * 0.02).to(bf)
+        stream, res = (torch.randn((rows, W), device=dev) for _ in range(2))
+        ones = torch.ones(W, device=dev)
+        inf = float("inf")
+
+        def routed(by_table):
+            if by_table:
+                chosen = ops.table_route(chosen_by, tokens)
+            else:
+                chosen, weights = ops.router_topk(x, router, top, scored=True)
+            position = None
+            if chosen.numel() <= ops.EXPERT_ROWS_ENTRIES:
+                results = ops.expert_rows_second(ops.expert_rows_first(x, w_gate_up[0], w_gate_up[1], chosen, inf, 1.0, 0.0), w_down, chosen)
+            elif chosen.numel() >= ops.GROUPED_ROWS_PER_EXPERT * E:
+                plan = ops.route_pad(chosen, E)
+                results = ops.grouped_second_product(ops.grouped_first_product(ops.gather_rows(x, plan), w_gate_up, plan, inf, 1.0, 0.0), w_down, plan)
+                position = plan.position
+            else:
+                plan = ops.route_sort(chosen, E)
+                results = ops.expert_second_product(ops.expert_first_product(x, w_gate_up[0], w_gate_up[1], plan, inf, 1.0, up_offset=0.0), w_down, plan)
+            if by_table:  # the entries' sum, the norm on it and the addition are one kernel
+                return ops.result_tanh_add(stream, results, 0.5, ones, ones, "rows", bf, top=top, position=position, entry_weight=1.0 / top)
+            return ops.outnorm_add(stream, ops.expert_combine(results, weights, position=position), ones, ones, 1e-6, copy_dtype=bf)
+
+        touched = min(E, rows * top)
+        for title, by_table in (("table_experts_and_add", True), ("scored_experts_and_add_rolevik", False)):
+            us = time_kernel(lambda: routed(by_table))
+            out[f"{name}_{title}"] = rated(us, flops=rows * top * 6 * W * F) if q_len > 1 else rated(us, moved=touched * 3 * W * F * 2)
+        # the norms on a result with the addition and the next reader's rows; beside Rolevik's
+        us = time_kernel(lambda: ops.result_tanh_add(stream, res, 0.5, ones, ones, (0.5, ones, ones), bf))
+        out[f"{name}_tanh_add_tanh"] = rated(us, moved=rows * W * (4 + 8 + 2))
+        us = time_kernel(lambda: ops.result_rms_add(stream, res, ones, 1e-6, (0.5, ones, ones), bf))
+        out[f"{name}_rms_add_tanh"] = rated(us, moved=rows * W * (4 + 8 + 2))
+        us = time_kernel(lambda: ops.outnorm_add(stream, res, ones, ones, 1e-6, copy_dtype=bf))
+        out[f"{name}_result_norm_add_rolevik"] = rated(us, moved=rows * W * (4 + 8 + 2))
+    return out
+
+
 def design_run(args) -> int:
     import torch
 
@@ -1019,6 +1216,10 @@ def design_run(args) -> int:
         title, all_sizes, make, params, beside, alone = "Rolevik", ROLEVIK_SIZES, rolevik_config, rolevik_layer_params, \
             kivezen_of_equal_size, rolevik_kernels
         other, other_title = "kivezen", "Kivezen of equal size (the parameters a token uses; one residual stream)"
+    elif args.design == "mabivik":
+        title, all_sizes, make, params, beside, alone = "Mabivik", MABIVIK_SIZES, mabivik_config, mabivik_layer_params, \
+            rolevik_of_equal_size, mabivik_kernels
+        other, other_title = "rolevik", "Rolevik of equal size (the parameters a token uses)"
     else:
         title, all_sizes, make, params, beside, alone = "Lovurax", LOVURAX_SIZES, lovurax_config, lovurax_layer_params, \
             (lambda z: llama_of_equal_size(z, lovurax_layer_params(z))), lovurax_kernels
@@ -1037,7 +1238,7 @@ def design_run(args) -> int:
             if arch == "llama":
                 entry[arch]["intermediate_size"] = config["intermediate_size"]
             elif arch == other:
-                entry[arch]["ff"] = config["layers"][0]["mlp"]["ff"]
+                entry[arch]["ff"] = next(layer["mlp"]["ff"] for layer in config["layers"] if layer["mlp"]["kind"] == "dense")
             model.close()
             del model
             torch.cuda.empty_cache()
@@ -1067,8 +1268,8 @@ def main() -> int:
     parser.add_argument("--only-prefill", action="store_true",
                         help="run the workload's prefill alone and print its figures (for profiling)")
     parser.add_argument("--size", default=None, choices=["s", "m"], help="with --design: one of its two sizes alone")
-    parser.add_argument("--design", default=None, choices=["kabanex", "lovurax", "kivezen", "rolevik"],
-                        help="instead of the default run: this design beside a model of equal size (a Llama; for kivezen a Lovurax, for rolevik a Kivezen): "
+    parser.add_argument("--design", default=None, choices=["kabanex", "lovurax", "kivezen", "rolevik", "mabivik"],
+                        help="instead of the default run: this design beside a model of equal size (a Llama; for kivezen a Lovurax, for rolevik a Kivezen, for mabivik a Rolevik): "
                              "prefill, decode, its kernels alone")
     args = parser.parse_args()
     if args.design and args.impl == "ours":

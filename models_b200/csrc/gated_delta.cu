@@ -31,10 +31,10 @@ __device__ __forceinline__ float softplus(float v) { return fmaxf(v, 0.0f) + log
 // taps - 1 inputs, from the step's tokens and, where the step brought fewer, from the old tail), so that no second kernel is
 // needed.  `split` (or null): the results also as two bfloat16 numbers each, rounding and rest, block by block of `per`
 // channels: [token][block][rounding of the block's channels | rests], what a tensor-core product with float-like accuracy reads.
-template <typename T>
+template <typename T, typename O>
 __global__ void __launch_bounds__(128)
 short_conv_kernel(const T* __restrict__ in, int in_stride, const float* __restrict__ in_bias, const float* __restrict__ weights,
-                  const float* __restrict__ out_bias, int activation, float* __restrict__ out, int out_stride,
+                  const float* __restrict__ out_bias, int activation, O* __restrict__ out, int out_stride,
                   float* __restrict__ state, size_t state_stride, const int* __restrict__ slots, const int* __restrict__ cu_q,
                   int channels, int taps, int store_tail, __nv_bfloat16* __restrict__ split, int per) {
     grid_launch_dependents();
@@ -74,7 +74,7 @@ short_conv_kernel(const T* __restrict__ in, int in_stride, const float* __restri
         for (int i = kMaxTaps - 1; i >= 0; --i) sum = fmaf(w[i], x[i], sum);  // oldest input first
         sum += bias_out;
         if (activation == 1) sum = sum * sigmoid(sum);
-        out[(size_t)(first + j) * out_stride + c] = sum;
+        Num<O>::store(out + (size_t)(first + j) * out_stride + c, sum);
         if (split != nullptr) {
             const __nv_bfloat16 rounding = __float2bfloat16_rn(sum);
             __nv_bfloat16* row = split + (size_t)(first + j) * 2 * channels + (size_t)(c / per) * 2 * per + c % per;
@@ -338,12 +338,12 @@ int pick_delta_walk(const float* conv, int conv_stride, const void* a_in, const 
 
 using namespace mb;
 
-// out [tokens, channels] float (row stride out_stride) = the convolution of the step's rows `in` (storage type, row stride
+// out [tokens, channels] (float, or bfloat16 where out_dtype says so and the inputs are; row stride out_stride) = the convolution of the step's rows `in` (storage type, row stride
 // in_stride) continued from every sequence's stored tail: state + slots[seq] * state_stride is [taps - 1][channels] floats.
 // activation: 0 none, 1 silu.  store_tail != 0: the new tail is stored too (0: the state is left as it is).
 // split (or null): bfloat16 [tokens][channels / per][2 * per], every result as its rounding and the rest.
 MB_EXPORT int mb_short_conv(const void* in, int in_stride, int dtype, const float* in_bias, const float* weights, const float* out_bias,
-                            int activation, float* out, int out_stride, float* state, size_t state_stride, const int* slots,
+                            int activation, void* out, int out_stride, int out_dtype, float* state, size_t state_stride, const int* slots,
                             const int* cu_q, int sequences, int max_q_len, int channels, int taps, int store_tail, void* split, int per,
                             cudaStream_t stream) {
     if (sequences <= 0 || max_q_len <= 0 || channels <= 0) return 0;
@@ -352,16 +352,15 @@ MB_EXPORT int mb_short_conv(const void* in, int in_stride, int dtype, const floa
     if (split != nullptr && (per <= 0 || channels % per)) return fail("short_conv: %d channels are no whole blocks of %d", channels, per);
     const dim3 grid((channels + 127) / 128, (max_q_len + kConvTokens - 1) / kConvTokens, sequences);
     if (grid.y > 65535) return fail("short_conv: a step of %d tokens per sequence exceeds the grid", max_q_len);
-    if (dtype == MB_F32)
-        MB_LAUNCH("short_conv", short_conv_kernel<float>, dim3(grid), dim3(128), 0, stream, true, (const float*)in, in_stride, in_bias,
-                  weights, out_bias, activation, out, out_stride, state, state_stride, slots, cu_q, channels, taps, store_tail,
-                  (__nv_bfloat16*)split, per);
-    else if (dtype == MB_BF16)
-        MB_LAUNCH("short_conv", short_conv_kernel<__nv_bfloat16>, dim3(grid), dim3(128), 0, stream, true, (const __nv_bfloat16*)in,
-                  in_stride, in_bias, weights, out_bias, activation, out, out_stride, state, state_stride, slots, cu_q, channels, taps,
-                  store_tail, (__nv_bfloat16*)split, per);
-    else
-        return fail("short_conv: unknown dtype code %d", dtype);
+#define MB_CONV(T, O)                                                                                                                  \
+    MB_LAUNCH("short_conv", (short_conv_kernel<T, O>), dim3(grid), dim3(128), 0, stream, true, (const T*)in, in_stride, in_bias, weights, \
+              out_bias, activation, (O*)out, out_stride, state, state_stride, slots, cu_q, channels, taps, store_tail,                  \
+              (__nv_bfloat16*)split, per)
+    if (dtype == MB_F32 && out_dtype == MB_F32) MB_CONV(float, float);
+    else if (dtype == MB_BF16 && out_dtype == MB_F32) MB_CONV(__nv_bfloat16, float);
+    else if (dtype == MB_BF16 && out_dtype == MB_BF16) MB_CONV(__nv_bfloat16, __nv_bfloat16);
+    else return fail("short_conv: dtype codes %d and %d are not built together", dtype, out_dtype);
+#undef MB_CONV
     return check_launch("short_conv");
 }
 

@@ -184,7 +184,8 @@ int pick_walk(int state, Args... args) {
     if (state <= 64) return launch_walk<T, R, 8>(args...);
     if (state <= 128) return launch_walk<T, R, 16>(args...);
     if (state <= 256) return launch_walk<T, R, 32>(args...);
-    return fail("state_space_walk: a state of %d rows per head exceeds 256", state);
+    if (state <= 512) return launch_walk<T, R, 64>(args...);  // (the registers overflow into local memory: correct, not fast)
+    return fail("state_space_walk: a state of %d rows per head exceeds 512", state);
 }
 
 template <typename T, typename Y>

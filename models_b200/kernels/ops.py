@@ -1135,10 +1135,11 @@ def _state_rows(state: torch.Tensor, offset: int, floats: int, name: str):
 
 def short_conv(x: torch.Tensor, weights: torch.Tensor, state: torch.Tensor, state_offset: int, slots: torch.Tensor, cu_q: torch.Tensor,
                max_q_len: int, in_bias: Optional[torch.Tensor] = None, out_bias: Optional[torch.Tensor] = None,
-               activation: Optional[str] = None, store_tail: bool = False, split_per: int = 0):
+               activation: Optional[str] = None, store_tail: bool = False, split_per: int = 0,
+               out_dtype: torch.dtype = torch.float32):
     """A short causal convolution over time per channel: with x_t = x[t] (+ in_bias) and `weights` [channels, taps] whose last
-    column meets the current token, out[t] = act(sum_i weights[:, taps - 1 - i] * x_(t - i) (+ out_bias)) as float32
-    [tokens, channels].  The inputs before a step's first token come from the sequence's tail, [taps - 1, channels] float32 at
+    column meets the current token, out[t] = act(sum_i weights[:, taps - 1 - i] * x_(t - i) (+ out_bias)) as `out_dtype`
+    [tokens, channels] (float arithmetic; rows that start on 16 bytes).  The inputs before a step's first token come from the sequence's tail, [taps - 1, channels] float32 at
     `state_offset` floats into its row of `state` (zeros for a new sequence); with `store_tail` the new tail is stored by the
     same kernel (else the state is left as it is).  `split_per` n > 0: also returns the results as two bfloat16 numbers
     each (the rounding and the rest), block by block of n channels, [tokens, channels / n * 2 n] with a block's roundings before
@@ -1156,13 +1157,13 @@ def short_conv(x: torch.Tensor, weights: torch.Tensor, state: torch.Tensor, stat
     if activation not in CONV_ACTIVATIONS:
         raise KernelError(f"short_conv: activation {activation!r} is not built (known: silu or none)")
     tail, stride = _state_rows(state, state_offset, (taps - 1) * channels, "short_conv")
-    out = torch.empty((x.shape[0], channels), dtype=torch.float32, device=x.device)
+    out = torch.empty((x.shape[0], -(-channels // 8) * 8), dtype=out_dtype, device=x.device)[:, :channels]
     if split_per and (split_per < 0 or channels % split_per):
         raise KernelError(f"short_conv: {channels} channels are no whole blocks of {split_per}")
     split = torch.empty((x.shape[0], 2 * channels), dtype=torch.bfloat16, device=x.device) if split_per else None
     lib = gated_delta_library()
     _run(lib, lib.mb_short_conv(_p(x), x.stride(0), _code(x.dtype), _p(in_bias), _p(weights), _p(out_bias), CONV_ACTIVATIONS[activation],
-                                _p(out), out.stride(0), tail, stride, _p(slots), _p(cu_q), cu_q.numel() - 1, max_q_len, channels, taps,
+                                _p(out), out.stride(0), _code(out_dtype), tail, stride, _p(slots), _p(cu_q), cu_q.numel() - 1, max_q_len, channels, taps,
                                 1 if store_tail else 0, _p(split), int(split_per), _stream()))
     return (out, split) if split_per else out
 
@@ -1227,6 +1228,47 @@ def state_space_walk(rows: torch.Tensor, x_at: int, b_at: int, c_at: int, dt_in:
     _run(lib, lib.mb_state_space_walk(_p(rows), rows.stride(0), _code(rows.dtype), _p(dt_in), dt_in.stride(0), _code(dt_in.dtype), _p(decay),
                                       _p(dt_bias), _p(skip), at, stride, _p(slots), _p(cu_q), cu_q.numel() - 1, _p(y), heads, groups,
                                       state_rows, vdim, x_at, b_at, c_at, _stream()))
+    return y
+
+
+def state_space_chunks_library(state_rows: int, vdim: int):
+    """The form for long steps, compiled for these sizes of a head's state at first use."""
+    return load_library("mb_state_space_chunks", ["state_space_chunks.cu"], {"MB_STATE": int(state_rows), "MB_VALUE_DIM": int(vdim)})
+
+
+SPACE_CHUNK_MIN_ROWS = 32  # steps that bring fewer tokens to every sequence are walked token by token
+
+
+def state_space_chunks_takes(dtype: torch.dtype, state_rows: int, vdim: int, max_q_len: int, groups_at: int) -> bool:
+    """bfloat16 steps of many tokens with state sizes that are multiples of 16 (rows up to 256, columns up to 128); `groups_at`:
+    the column where B starts."""
+    return (dtype == torch.bfloat16 and max_q_len >= SPACE_CHUNK_MIN_ROWS and state_rows % 16 == 0 and vdim % 16 == 0
+            and state_rows <= 256 and vdim <= 128 and groups_at % 8 == 0)
+
+
+def state_space_chunks(rows: torch.Tensor, x_at: int, b_at: int, c_at: int, dt_in: torch.Tensor, decay: torch.Tensor, dt_bias: torch.Tensor,
+                       skip: torch.Tensor, state: torch.Tensor, state_offset: int, slots: torch.Tensor, cu_q: torch.Tensor, max_q_len: int,
+                       heads: int, groups: int, state_rows: int, vdim: int) -> torch.Tensor:
+    """What state_space_walk computes, for long steps in bfloat16 (`rows`, dt_in and the result): chunks of 128 tokens on the tensor
+    cores, the states at the chunks' borders carried in float."""
+    _cuda(rows, dt_in, decay, dt_bias, skip, state, slots, cu_q)
+    _int32(slots, "slots")
+    _int32(cu_q, "cu_q")
+    _state_space_checks("state_space_chunks", rows, x_at, b_at, c_at, dt_in, decay, dt_bias, skip, heads, groups, state_rows, vdim)
+    if rows.dtype != torch.bfloat16 or dt_in.dtype != torch.bfloat16:
+        raise KernelError("state_space_chunks: the convolved rows and the step sizes must be bfloat16")
+    at, stride = _state_rows(state, state_offset, heads * state_rows * vdim, "state_space_chunks")
+    tokens, sequences, device = rows.shape[0], cu_q.numel() - 1, rows.device
+    lib = state_space_chunks_library(state_rows, vdim)
+    places = tokens // lib.mb_state_space_chunk_tokens() + sequences
+    y = torch.empty((tokens, heads * vdim), dtype=torch.bfloat16, device=device)
+    added = torch.empty((places, heads, state_rows * vdim), dtype=torch.float32, device=device)
+    starts = torch.empty((2, places, heads, state_rows * vdim), dtype=torch.bfloat16, device=device)
+    keep = torch.empty((places, heads), dtype=torch.float32, device=device)
+    _run(lib, lib.mb_state_space_chunks(_p(rows), rows.stride(0), _p(dt_in), dt_in.stride(0), _p(decay), _p(dt_bias), _p(skip), at, stride,
+                                        _p(slots), _p(cu_q), sequences, max_q_len, _p(y), _p(added), _p(starts[0]), _p(starts[1]), _p(keep),
+                                        heads, groups, x_at, b_at, c_at, _stream()))
+    _launches[0] += 2  # three kernels
     return y
 
 

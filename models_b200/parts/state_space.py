@@ -79,10 +79,16 @@ class StateSpaceMixer(SplitPart, Mixer):
         z, xbc, dt = proj[:, at[0]:at[0] + inner], proj[:, at[1]:at[1] + self.channels], proj[:, at[2]:at[2] + H]
         b_at = inner
         c_at = inner + s.groups * s.state_size
+        chunked = ops.state_space_chunks_takes(proj.dtype, s.state_size, s.value_dim, batch.max_q_len, b_at)
         conv = ops.short_conv(xbc, self.conv, run.state, self.state_floats, batch.slots, batch.cu_q, batch.max_q_len,
-                              out_bias=self.conv_bias, activation="silu", store_tail=True)
-        y = ops.state_space_walk(conv, 0, b_at, c_at, dt, self.decay, self.dt_bias, self.skip, run.state, 0, batch.slots, batch.cu_q, H,
-                                 s.groups, s.state_size, s.value_dim)
+                              out_bias=self.conv_bias, activation="silu", store_tail=True,
+                              out_dtype=torch.bfloat16 if chunked else torch.float32)
+        sizes = (H, s.groups, s.state_size, s.value_dim)
+        if chunked:
+            y = ops.state_space_chunks(conv, 0, b_at, c_at, dt, self.decay, self.dt_bias, self.skip, run.state, 0, batch.slots, batch.cu_q,
+                                       batch.max_q_len, *sizes)
+        else:
+            y = ops.state_space_walk(conv, 0, b_at, c_at, dt, self.decay, self.dt_bias, self.skip, run.state, 0, batch.slots, batch.cu_q, *sizes)
         ops.gate_part_norm(y, z, self.gain, s.eps, s.norm_groups, mid, scale)
 
 
