@@ -345,7 +345,8 @@ __global__ void project_norm_rotate_store_kernel(T* __restrict__ q, int q_stride
     }
 }
 
-// grid (tokens); block 128.  What a latent attention does to the rows of its first product: the query's latent (q_width numbers,
+// grid (tokens, 2); block 128 (block 0 of a token: the query's latent; block 1: the cached row).  What a latent attention does to
+// the rows of its first product: the query's latent (q_width numbers,
 // null: none) divided by its root mean square and multiplied by its gain, into rows of its own that are zero up to q_columns;
 // and the row the cache keeps, [latent | tail]: the latent normalised the same way with its own gain, the tail's `turned`
 // numbers rotated by the token's position (pairs (i, i + turned / 2), tables [positions][turned / 2]).  k null: no row is stored.
@@ -359,7 +360,8 @@ latent_prepare_kernel(const T* __restrict__ q, int q_stride, const float* __rest
     grid_dependency_wait();
     __shared__ float scratch[32];
     const size_t token = blockIdx.x;
-    if (q != nullptr) {
+    if (blockIdx.y == 0) {
+        if (q == nullptr) return;
         const T* src = q + token * q_stride;
         float squares = 0.0f;
         for (int i = threadIdx.x; i < q_width; i += blockDim.x) {
@@ -369,6 +371,7 @@ latent_prepare_kernel(const T* __restrict__ q, int q_stride, const float* __rest
         const float factor = 1.0f / sqrtf(block_sum(squares, scratch) / (float)q_width + eps);
         for (int i = threadIdx.x; i < q_columns; i += blockDim.x)
             Num<T>::store(q_out + token * q_columns + i, i < q_width ? Num<T>::load(src + i) * factor * q_gain[i] : 0.0f);
+        return;
     }
     if (k == nullptr) return;
     const int slot = slot_mapping[token];
@@ -869,6 +872,7 @@ head_linear_tc_kernel(const bf16* __restrict__ in, int in_stride, const bf16* __
     const int head = blockIdx.y, first = blockIdx.x * kTile;
     const int valid = min(kTile, tokens - first);
     const bf16* w_head = w + (size_t)head * n_out * n_in;
+    const bool gate_in_twos = gate_stride % 2 == 0 && !((uintptr_t)gate & 3);
     const uint32_t x_tile = smem_u32(tc_smem), w_tiles = x_tile + tile_bytes;
     const int chunks = (n_out + kTile - 1) / kTile;
     auto load_weights = [&](int chunk, int stage) {
@@ -886,7 +890,21 @@ head_linear_tc_kernel(const bf16* __restrict__ in, int in_stride, const bf16* __
         if (row < valid) v = *reinterpret_cast<const uint4*>(in + (size_t)(first + row) * in_stride + (size_t)head * layout.in_head + piece * 8);
         *reinterpret_cast<uint4*>(tc_smem + row * row_bytes + piece * 16) = v;
     }
-    if (layout.turned > 0) {
+    if (layout.turned > 0 && layout.turned % 4 == 0) {  // two neighbouring pairs at a time
+        const int half = layout.turned / 2, quarter = half / 2;
+        for (int item = threadIdx.x; item < valid * quarter; item += 128) {
+            const size_t row = first + item / quarter;
+            const int pair = item % quarter * 2;
+            const bf16* src = in + row * in_stride + (size_t)head * layout.in_head + n_in + pair;
+            bf16* dst = out + row * out_stride + (size_t)head * layout.out_head + n_out + pair;
+            const size_t at = (size_t)layout.positions[row] * half + pair;
+            const float2 c = *reinterpret_cast<const float2*>(layout.cos + at), s = *reinterpret_cast<const float2*>(layout.sin + at);
+            const float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(src));
+            const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(src + half));
+            *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(u.x * c.x - v.x * s.x, u.y * c.y - v.y * s.y);
+            *reinterpret_cast<__nv_bfloat162*>(dst + half) = __floats2bfloat162_rn(v.x * c.x + u.x * s.x, v.y * c.y + u.y * s.y);
+        }
+    } else if (layout.turned > 0) {
         const int half = layout.turned / 2;
         for (int item = threadIdx.x; item < valid * half; item += 128) {
             const size_t row = first + item / half;
@@ -931,10 +949,18 @@ head_linear_tc_kernel(const bf16* __restrict__ in, int in_stride, const bf16* __
                 bf16* dst = out + (size_t)(first + row) * out_stride + (size_t)head * layout.out_head + n;
                 if (gate != nullptr && layout.element_gate) {
                     const bf16* g = gate + (size_t)(first + row) * gate_stride + (size_t)head * n_out + n;
-                    s[0][2 * r] *= sigmoid(__bfloat162float(g[0]));
-                    s[0][2 * r + 1] *= sigmoid(__bfloat162float(g[1]));
-                    s[1][2 * r] *= sigmoid(__bfloat162float(g[8]));
-                    s[1][2 * r + 1] *= sigmoid(__bfloat162float(g[9]));
+                    float2 a, b;
+                    if (gate_in_twos) {
+                        a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(g));
+                        b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(g + 8));
+                    } else {
+                        a = make_float2(__bfloat162float(g[0]), __bfloat162float(g[1]));
+                        b = make_float2(__bfloat162float(g[8]), __bfloat162float(g[9]));
+                    }
+                    s[0][2 * r] *= sigmoid(a.x);
+                    s[0][2 * r + 1] *= sigmoid(a.y);
+                    s[1][2 * r] *= sigmoid(b.x);
+                    s[1][2 * r + 1] *= sigmoid(b.y);
                 }
                 *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(s[0][2 * r] * factor[r], s[0][2 * r + 1] * factor[r]);
                 *reinterpret_cast<__nv_bfloat162*>(dst + 8) = __floats2bfloat162_rn(s[1][2 * r] * factor[r], s[1][2 * r + 1] * factor[r]);
@@ -1258,11 +1284,11 @@ MB_EXPORT int mb_latent_prepare(const void* q, int q_stride, const float* q_gain
     if (q != nullptr && (q_width <= 0 || q_columns < q_width)) return fail("latent_prepare: %d query numbers in rows of %d", q_width, q_columns);
     if (k != nullptr && latent <= 0) return fail("latent_prepare: a latent of %d numbers", latent);
     if (dtype == MB_F32)
-        MB_LAUNCH("latent_prepare", latent_prepare_kernel<float>, dim3(tokens), dim3(128), 0, stream, true, (const float*)q, q_stride, q_gain,
+        MB_LAUNCH("latent_prepare", latent_prepare_kernel<float>, dim3(tokens, k != nullptr ? 2 : 1), dim3(128), 0, stream, true, (const float*)q, q_stride, q_gain,
                   q_width, (float*)q_out, q_columns, (const float*)k, k_stride, k_gain, latent, turned, cos, sin, positions, eps, (float*)k_pool,
                   slot_mapping);
     else if (dtype == MB_BF16)
-        MB_LAUNCH("latent_prepare", latent_prepare_kernel<__nv_bfloat16>, dim3(tokens), dim3(128), 0, stream, true, (const __nv_bfloat16*)q,
+        MB_LAUNCH("latent_prepare", latent_prepare_kernel<__nv_bfloat16>, dim3(tokens, k != nullptr ? 2 : 1), dim3(128), 0, stream, true, (const __nv_bfloat16*)q,
                   q_stride, q_gain, q_width, (__nv_bfloat16*)q_out, q_columns, (const __nv_bfloat16*)k, k_stride, k_gain, latent, turned, cos,
                   sin, positions, eps, (__nv_bfloat16*)k_pool, slot_mapping);
     else

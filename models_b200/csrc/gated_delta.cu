@@ -86,6 +86,77 @@ short_conv_kernel(const T* __restrict__ in, int in_stride, const float* __restri
     }
 }
 
+// The same with four neighbouring channels a thread (8- or 16-byte loads and stores): many tokens and channels in fours, nothing split.
+// grid (ceil(channels / 4 / 64), ceil(max_q_len / kConvTokens), sequences); block 64.
+template <typename T>
+__device__ __forceinline__ float4 load_four(const T* p);
+template <>
+__device__ __forceinline__ float4 load_four<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <>
+__device__ __forceinline__ float4 load_four<__nv_bfloat16>(const __nv_bfloat16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(raw.x << 16), __uint_as_float(raw.x & 0xffff0000u), __uint_as_float(raw.y << 16), __uint_as_float(raw.y & 0xffff0000u));
+}
+__device__ __forceinline__ void store_four(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store_four(__nv_bfloat16* p, float4 v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+__device__ __forceinline__ float4 add_four(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
+
+template <typename T, typename O, int kTaps>
+__global__ void __launch_bounds__(64)
+short_conv_fours_kernel(const T* __restrict__ in, int in_stride, const float* __restrict__ in_bias, const float* __restrict__ weights,
+                        const float* __restrict__ out_bias, int activation, O* __restrict__ out, int out_stride, float* __restrict__ state,
+                        size_t state_stride, const int* __restrict__ slots, const int* __restrict__ cu_q, int channels, int store_tail) {
+    grid_launch_dependents();
+    grid_dependency_wait();
+    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4, seq = blockIdx.z;
+    const int first = cu_q[seq], count = cu_q[seq + 1] - first;
+    const int j0 = blockIdx.y * kConvTokens, j1 = min(j0 + kConvTokens, count);
+    if (c >= channels || j0 >= count) return;
+    float* tail = state + (size_t)slots[seq] * state_stride;
+    const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    const float4 bias_in = in_bias != nullptr ? load_four<float>(in_bias + c) : zero, bias_out = out_bias != nullptr ? load_four<float>(out_bias + c) : zero;
+    float4 w[kTaps], x[kTaps];  // w[i] meets the input i tokens back; x[i] is that input
+    auto input = [&](int j) { return add_four(load_four<T>(in + (size_t)(first + j) * in_stride + c), bias_in); };
+    auto stored = [&](int row) { return make_float4(tail[(size_t)row * channels + c], tail[(size_t)row * channels + c + 1], tail[(size_t)row * channels + c + 2], tail[(size_t)row * channels + c + 3]); };
+#pragma unroll
+    for (int i = 0; i < kTaps; ++i) {
+        const float* at = weights + (size_t)c * kTaps + (kTaps - 1 - i);
+        w[i] = make_float4(at[0], at[kTaps], at[2 * kTaps], at[3 * kTaps]);
+        x[i] = zero;
+        if (i >= 1) x[i] = j0 >= i ? input(j0 - i) : stored(kTaps - 1 + j0 - i);
+    }
+    if (store_tail && j0 == 0) {
+#pragma unroll
+        for (int i = 0; i < kTaps - 1; ++i) {  // tail row i is the input of token count - (kTaps - 1) + i; a negative token is an old row, held in x
+            const int j = count - (kTaps - 1) + i;
+            float4 kept = zero;
+#pragma unroll
+            for (int back = 1; back < kTaps; ++back)
+                if (back == -j) kept = x[back];
+            if (j >= 0) kept = input(j);
+            float* dst = tail + (size_t)i * channels + c;
+            dst[0] = kept.x, dst[1] = kept.y, dst[2] = kept.z, dst[3] = kept.w;
+        }
+    }
+    for (int j = j0; j < j1; ++j) {
+        x[0] = input(j);
+        float4 sum = zero;
+#pragma unroll
+        for (int i = kTaps - 1; i >= 0; --i) {  // oldest input first
+            sum.x = fmaf(w[i].x, x[i].x, sum.x), sum.y = fmaf(w[i].y, x[i].y, sum.y);
+            sum.z = fmaf(w[i].z, x[i].z, sum.z), sum.w = fmaf(w[i].w, x[i].w, sum.w);
+        }
+        sum = add_four(sum, bias_out);
+        if (activation == 1) sum = make_float4(sum.x * sigmoid(sum.x), sum.y * sigmoid(sum.y), sum.z * sigmoid(sum.z), sum.w * sigmoid(sum.w));
+        store_four(out + (size_t)(first + j) * out_stride + c, sum);
+#pragma unroll
+        for (int i = kTaps - 1; i >= 1; --i) x[i] = x[i - 1];
+    }
+}
+
 struct DeltaShape {
     int heads, kv_heads, dim, vdim;
     int q_at, k_at, v_at;  // first columns of the convolved rows' q, k and v parts
@@ -356,6 +427,26 @@ MB_EXPORT int mb_short_conv(const void* in, int in_stride, int dtype, const floa
     MB_LAUNCH("short_conv", (short_conv_kernel<T, O>), dim3(grid), dim3(128), 0, stream, true, (const T*)in, in_stride, in_bias, weights, \
               out_bias, activation, (O*)out, out_stride, state, state_stride, slots, cu_q, channels, taps, store_tail,                  \
               (__nv_bfloat16*)split, per)
+    const size_t in_bytes = dtype == MB_F32 ? 4 : 2, out_bytes = out_dtype == MB_F32 ? 4 : 2;
+    if (split == nullptr && max_q_len > kConvTokens && channels % 4 == 0 && in_stride % 4 == 0 && out_stride % 4 == 0 && (taps == 2 || taps == 3 || taps == 4) &&
+        !((uintptr_t)in % (4 * in_bytes)) && !((uintptr_t)out % (4 * out_bytes)) && !((uintptr_t)in_bias & 15) && !((uintptr_t)out_bias & 15)) {
+        const dim3 fours((channels / 4 + 63) / 64, grid.y, sequences);
+#define MB_FOURS(T, O, TAPS)                                                                                                                \
+    MB_LAUNCH("short_conv", (short_conv_fours_kernel<T, O, TAPS>), fours, dim3(64), 0, stream, true, (const T*)in, in_stride, in_bias, weights, \
+              out_bias, activation, (O*)out, out_stride, state, state_stride, slots, cu_q, channels, store_tail)
+#define MB_FOURS_OF(T, O)                    \
+    do {                                     \
+        if (taps == 2) MB_FOURS(T, O, 2);      \
+        else if (taps == 3) MB_FOURS(T, O, 3); \
+        else MB_FOURS(T, O, 4);                \
+        return check_launch("short_conv");   \
+    } while (0)
+        if (dtype == MB_F32 && out_dtype == MB_F32) MB_FOURS_OF(float, float);
+        if (dtype == MB_BF16 && out_dtype == MB_F32) MB_FOURS_OF(__nv_bfloat16, float);
+        if (dtype == MB_BF16 && out_dtype == MB_BF16) MB_FOURS_OF(__nv_bfloat16, __nv_bfloat16);
+#undef MB_FOURS_OF
+#undef MB_FOURS
+    }
     if (dtype == MB_F32 && out_dtype == MB_F32) MB_CONV(float, float);
     else if (dtype == MB_BF16 && out_dtype == MB_F32) MB_CONV(__nv_bfloat16, float);
     else if (dtype == MB_BF16 && out_dtype == MB_BF16) MB_CONV(__nv_bfloat16, __nv_bfloat16);

@@ -494,15 +494,29 @@ expert_product_kernel(const T* __restrict__ a, int a_stride, const T* __restrict
 template <typename T, bool kFirst, bool kVector>
 __global__ void __launch_bounds__(256)
 expert_rows_kernel(const T* __restrict__ a, int a_stride, const T* __restrict__ w0, const T* __restrict__ w1, T* __restrict__ mid,
-                   float* __restrict__ slot_out, int out_stride, const int* __restrict__ chosen, int top, int experts, int N, int K,
-                   float limit, float slope, float up_offset) {
+                   float* __restrict__ slot_out, int out_stride, const int* __restrict__ chosen, const int* __restrict__ table_tokens,
+                   int top, int experts, int N, int K, float limit, float slope, float up_offset) {
     grid_launch_dependents();
-    grid_dependency_wait();
     constexpr int kCols = 4;
     constexpr int kSets = kFirst ? 2 : 1;
     extern __shared__ __align__(16) float rows_shared[];  // K floats
     const int entry = blockIdx.y;
-    const int expert = chosen[entry];
+    int expert = -1;
+    if (table_tokens != nullptr) {
+        // a table of token ids: neither it nor the ids come from a kernel of this step, so the expert is known and its weights are on
+        // their way into L2 while the kernels before this one still run
+        expert = chosen[(size_t)table_tokens[entry / top] * top + entry % top];
+        const int n0 = (blockIdx.x * 8 + (threadIdx.x >> 5)) * kCols;
+        if (expert >= 0 && expert < experts && n0 < N) {
+            const size_t row_bytes = (size_t)K * sizeof(T), bytes = row_bytes * min(kCols, N - n0), at = ((size_t)expert * N + n0) * row_bytes;
+            for (size_t b = (threadIdx.x & 31) * 128; b < bytes; b += 32 * 128) {
+                asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const unsigned char*>(w0) + at + b));
+                if (kFirst) asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const unsigned char*>(w1) + at + b));
+            }
+        }
+    }
+    grid_dependency_wait();
+    if (table_tokens == nullptr) expert = chosen[entry];
     if (expert < 0 || expert >= experts) return;  // (a router that chose nothing real: nothing is written)
     const T* src = a + (size_t)(kFirst ? entry / top : entry) * a_stride;
     if (kVector) {
@@ -945,9 +959,10 @@ MB_EXPORT int mb_expert_product(const void* a, int a_stride, const void* w0, con
 }
 
 // The products for few entries (see expert_rows_kernel); rows of mid and slot_out in entry order (token * top + choice).
+// table_tokens (or null): `chosen` is a table [vocab][top] and entry i's expert is chosen[table_tokens[i / top]][i % top].
 MB_EXPORT int mb_expert_rows(const void* a, int a_stride, const void* w0, const void* w1, void* mid, float* slot_out, int out_stride,
-                             int dtype, const int* chosen, int entries, int top, int experts, int N, int K, float limit, float slope, float up_offset,
-                             int first, cudaStream_t stream) {
+                             int dtype, const int* chosen, const int* table_tokens, int entries, int top, int experts, int N, int K, float limit,
+                             float slope, float up_offset, int first, cudaStream_t stream) {
     if (entries <= 0) return 0;
     if (N <= 0 || K <= 0 || top <= 0 || experts <= 0) return fail("expert_rows: N %d, K %d, top %d, %d experts", N, K, top, experts);
     if (entries > 65535) return fail("expert_rows: %d entries exceed the grid limit 65535", entries);
@@ -962,7 +977,7 @@ MB_EXPORT int mb_expert_rows(const void* a, int a_stride, const void* w0, const 
     do {                                                                                                                             \
         if (smem > 48 * 1024) cudaFuncSetAttribute(expert_rows_kernel<T, FIRST, VECTOR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         MB_LAUNCH("expert_rows", (expert_rows_kernel<T, FIRST, VECTOR>), grid, dim3(256), smem, stream, true, (const T*)a, a_stride,  \
-                  (const T*)w0, (const T*)w1, (T*)mid, slot_out, out_stride, chosen, top, experts, N, K, limit, slope, up_offset);               \
+                  (const T*)w0, (const T*)w1, (T*)mid, slot_out, out_stride, chosen, table_tokens, top, experts, N, K, limit, slope, up_offset); \
     } while (0)
 #define MB_ROWS_OF(T)                                                              \
     do {                                                                           \

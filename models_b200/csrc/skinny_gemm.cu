@@ -48,7 +48,7 @@ namespace mb {
 using bf16 = __nv_bfloat16;
 
 enum { PRO_NONE = 0, PRO_NORM = 1, PRO_PRE = 2 };
-enum { EPI_BF16 = 0, EPI_F32 = 1, EPI_RESIDUAL = 2, EPI_SWIGLU = 3, EPI_ROPE = 4 };
+enum { EPI_BF16 = 0, EPI_F32 = 1, EPI_RESIDUAL = 2, EPI_SWIGLU = 3, EPI_ROPE = 4, EPI_TANH = 5, EPI_SIDE = 6 };
 
 constexpr int kWarps = 4;
 constexpr int kThreads = kWarps * 32;
@@ -110,6 +110,21 @@ struct SkinnyArgs {
     const bf16* gate;         // [batch][ld_gate]
     int ld_gate;
     const float* gate_bias;   // [n]
+    // EPI_TANH: the residual stream gets tanh(tanh_alpha * result) * tanh_weight + tanh_bias; its new row is then left for the next
+    // reader as it is (then_kind 1) or through that reader's own tanh(then_alpha * .) * then_weight + then_bias (2)
+    float tanh_alpha;
+    const float* tanh_weight;  // [n]
+    const float* tanh_bias;
+    int then_kind;
+    float then_alpha;
+    const float* then_weight;
+    const float* then_bias;
+    bf16* then_rows;           // [batch][ld_then]
+    int ld_then;
+    // EPI_SIDE: out_bf16 = gelu_tanh(result) * side_table[side_tokens[b]][row] for row < side_dim, 0 behind
+    const bf16* side_table;    // [vocab][side_dim]
+    const int* side_tokens;    // [batch]
+    int side_dim;
     const int* rows;      // optional: activation row b is xf row rows[b]
     bf16* out_bf16;
     float* out_f32;       // EPI_F32 output, or the residual stream for EPI_RESIDUAL
@@ -229,7 +244,8 @@ skinny_gemm_kernel(const SkinnyArgs args) {
     // step began) and weights -- the position, cache slot, cosine and sine of this thread's first finishing item, the next
     // norm's gain for it, and this norm's gain on its way into L2.
     int my_position = 0, my_slot = -1;   // EPI_ROPE: of the batch column of this thread's first finishing item
-    float first_a = 0.0f, first_b = 0.0f;  // EPI_ROPE: its cosine and sine in the first row tile; EPI_RESIDUAL: the next norm's gain
+    float first_a = 0.0f, first_b = 0.0f;  // EPI_ROPE: its cosine and sine in the first row tile; EPI_RESIDUAL: the next norm's gain; EPI_TANH: the norm's weight and bias
+    float then_w = 0.0f, then_b = 0.0f;    // EPI_TANH: the next reader's
     {
         const int row_in_tile = threadIdx.x % kTileRows, col = threadIdx.x / kTileRows;
         if (EPI == EPI_ROPE && col < args.batch) {
@@ -240,6 +256,15 @@ skinny_gemm_kernel(const SkinnyArgs args) {
                 const size_t at_table = (size_t)my_position * (args.head_dim / 2) + (cluster_id % tiles_per_head) * 8 + row_in_tile;
                 first_a = args.cos_table[at_table];
                 first_b = args.sin_table[at_table];
+            }
+        }
+        if (EPI == EPI_TANH && tiles_mine > 0 && cluster_id * kTileRows + row_in_tile < rows_total) {
+            const int row = cluster_id * kTileRows + row_in_tile;
+            first_a = args.tanh_weight[row];
+            first_b = args.tanh_bias[row];
+            if (args.then_kind == 2) {
+                then_w = args.then_weight[row];
+                then_b = args.then_bias[row];
             }
         }
         if (EPI == EPI_RESIDUAL && args.emit_gain != nullptr && tiles_mine > 0 && cluster_id * kTileRows + row_in_tile < rows_total)
@@ -382,7 +407,9 @@ skinny_gemm_kernel(const SkinnyArgs args) {
             const int row_in_tile = threadIdx.x % kTileRows, col = threadIdx.x / kTileRows;
             const int row = tile * kTileRows + row_in_tile;
             if (rank == 0 && row < rows_total && col < args.batch) {
-                if (EPI == EPI_RESIDUAL) early_a = args.out_f32[(size_t)col * args.ld_out + row];
+                if (EPI == EPI_RESIDUAL || EPI == EPI_TANH) early_a = args.out_f32[(size_t)col * args.ld_out + row];
+                if (EPI == EPI_SIDE && row < args.side_dim)
+                    early_a = __bfloat162float(args.side_table[(size_t)args.side_tokens[col] * args.side_dim + row]);
                 if (EPI == EPI_ROPE) {
                     const int tiles_per_head = args.head_dim / 16;
                     if (local == 0) {
@@ -455,6 +482,23 @@ skinny_gemm_kernel(const SkinnyArgs args) {
                     args.emit_rows[(size_t)col * args.ld_emit + row] = __float2bfloat16_rn(x_new * gain);
                     squares = x_new * x_new;
                 }
+            }
+            if (EPI == EPI_TANH) {
+                const bool early = i == (int)threadIdx.x;
+                const bool held = early && local == 0;
+                const float w = held ? first_a : args.tanh_weight[row], b = held ? first_b : args.tanh_bias[row];
+                const float x_new = (early ? early_a : args.out_f32[at]) + fmaf(tanhf(args.tanh_alpha * value), w, b);
+                args.out_f32[at] = x_new;
+                if (args.then_kind != 0) {
+                    const float next = args.then_kind == 1 ? x_new
+                        : fmaf(tanhf(args.then_alpha * x_new), held ? then_w : args.then_weight[row], held ? then_b : args.then_bias[row]);
+                    args.then_rows[(size_t)col * args.ld_then + row] = __float2bfloat16_rn(next);
+                }
+            }
+            if (EPI == EPI_SIDE) {
+                float e = early_a;
+                if (i != (int)threadIdx.x) e = row < args.side_dim ? __bfloat162float(args.side_table[(size_t)args.side_tokens[col] * args.side_dim + row]) : 0.0f;
+                args.out_bf16[at] = __float2bfloat16_rn(row < args.side_dim ? gate_activation(MB_ACT_GELU_TANH, value) * e : 0.0f);
             }
             if (EPI == EPI_SWIGLU) args.out_bf16[at] = __float2bfloat16_rn(gate_activation(args.activation, value) * second);
             if (EPI == EPI_ROPE) {
@@ -622,6 +666,8 @@ static int skinny_gemm(const void* w, int ldw, int n, int k, int batch, const vo
     MB_CASE(PRO_PRE, EPI_F32)
     MB_CASE(PRO_PRE, EPI_SWIGLU)
     MB_CASE(PRO_PRE, EPI_ROPE)
+    MB_CASE(PRO_NONE, EPI_TANH)
+    MB_CASE(PRO_NONE, EPI_SIDE)
 #undef MB_CASE
     return fail("skinny_gemm: no kernel for prologue %d with epilogue %d", prologue, epilogue);
 }
@@ -636,7 +682,7 @@ MB_EXPORT int mb_skinny_gemm(const void* w, int ldw, int n, int k, int batch, co
                              int epilogue, int multiprocessors, int dependent, const float* ssq_parts, int ssq_count,
                              const float* emit_gain, void* emit_rows, int ld_emit, float* emit_ssq, int* parts_written,
                              cudaStream_t stream) {
-    if ((epilogue & 0xff) == EPI_ROPE) return fail("skinny_gemm: the rotary epilogue has an entry point of its own");
+    if ((epilogue & 0xff) >= EPI_ROPE) return fail("skinny_gemm: epilogue %d has an entry point of its own", epilogue & 0xff);
     SkinnyArgs args{};
     args.ssq_parts = ssq_parts; args.ssq_count = ssq_count;
     args.emit_gain = emit_gain; args.emit_rows = (bf16*)emit_rows; args.ld_emit = ld_emit; args.emit_ssq = emit_ssq;
@@ -655,6 +701,32 @@ MB_EXPORT int mb_skinny_gemm_gated_residual(const void* w, int ldw, int n, int k
     args.gate = (const bf16*)gate; args.ld_gate = ld_gate; args.gate_bias = gate_bias;
     return skinny_gemm(w, ldw, n, k, batch, x, ldx, nullptr, 0, nullptr, 0.0f, nullptr, out, ld_out, EPI_RESIDUAL, multiprocessors,
                        dependent, args, stream);
+}
+
+// x_out += tanh(alpha * (x . w^T)) * weight + bias (weight, bias: float [n]); the new rows are then left in then_rows (bfloat16, row
+// stride ld_then) as they are (then_kind 1) or as tanh(then_alpha * .) * then_weight + then_bias (2).
+MB_EXPORT int mb_skinny_gemm_tanh_residual(const void* w, int ldw, int n, int k, int batch, const void* x, int ldx, void* out, int ld_out,
+                                           float alpha, const float* weight, const float* bias, int then_kind, float then_alpha,
+                                           const float* then_weight, const float* then_bias, void* then_rows, int ld_then,
+                                           int multiprocessors, int dependent, cudaStream_t stream) {
+    if (!weight || !bias || then_kind < 0 || then_kind > 2 || (then_kind != 0 && !then_rows) || (then_kind == 2 && (!then_weight || !then_bias)))
+        return fail("skinny_gemm_tanh_residual: the norm or what follows (%d) lacks its tensors", then_kind);
+    SkinnyArgs args{};
+    args.tanh_alpha = alpha; args.tanh_weight = weight; args.tanh_bias = bias;
+    args.then_kind = then_kind; args.then_alpha = then_alpha; args.then_weight = then_weight; args.then_bias = then_bias;
+    args.then_rows = (bf16*)then_rows; args.ld_then = ld_then;
+    return skinny_gemm(w, ldw, n, k, batch, x, ldx, nullptr, 0, nullptr, 0.0f, nullptr, out, ld_out, EPI_TANH, multiprocessors, dependent,
+                       args, stream);
+}
+
+// out [batch, n] bfloat16 = gelu_tanh(x . w^T) * table[token] for columns below dim (table bfloat16 [vocab][dim]), 0 behind them.
+MB_EXPORT int mb_skinny_gemm_side(const void* w, int ldw, int n, int k, int batch, const void* x, int ldx, void* out, int ld_out,
+                                  const void* table, const int* tokens, int dim, int multiprocessors, int dependent, cudaStream_t stream) {
+    if (!table || !tokens || dim <= 0 || dim > n) return fail("skinny_gemm_side: a table of %d columns for %d outputs", dim, n);
+    SkinnyArgs args{};
+    args.side_table = (const bf16*)table; args.side_tokens = tokens; args.side_dim = dim;
+    return skinny_gemm(w, ldw, n, k, batch, x, ldx, nullptr, 0, nullptr, 0.0f, nullptr, out, ld_out, EPI_SIDE, multiprocessors, dependent,
+                       args, stream);
 }
 
 // The q/k/v product of an attention layer with rotation and cache write folded in.  w: [(heads + 2 *

@@ -120,43 +120,76 @@ __global__ void space_walk_kernel(const R* __restrict__ rows, int row_stride, co
     }
 }
 
-// grid (tokens, parts); block 128 or 256.  Rows whose parts fit stay in registers between the sum and the store.
-template <typename T, typename Y, int kKept>
-__global__ void gate_part_norm_kernel(const Y* __restrict__ y, const T* __restrict__ z, int z_stride, const float* __restrict__ gain, float eps,
-                                      T* __restrict__ out, int out_stride, float out_scale, int width, int size) {
+// grid (tokens, parts); block a multiple of 32.  kVec neighbouring numbers a thread and step (8: 16-byte loads of bfloat16 rows); the
+// first kKept steps' products stay in registers between the sum and the store, parts larger than that are read twice.
+template <typename T, int kVec>
+__device__ __forceinline__ void load_some(const T* p, float (&v)[kVec]) {
+    if constexpr (kVec == 8) {
+        load8(p, v);
+    } else {
+#pragma unroll
+        for (int j = 0; j < kVec; ++j) v[j] = Num<T>::load(p + j);
+    }
+}
+
+template <typename T, typename Y, int kVec, int kKept>
+__global__ void __launch_bounds__(256)
+gate_part_norm_kernel(const Y* __restrict__ y, const T* __restrict__ z, int z_stride, const float* __restrict__ gain, float eps,
+                      T* __restrict__ out, int out_stride, float out_scale, int width, int size) {
     grid_launch_dependents();
     grid_dependency_wait();
     __shared__ float scratch[32];
     const size_t token = blockIdx.x;
-    const int at = blockIdx.y * size;
+    const int at = blockIdx.y * size, step = blockDim.x * kVec;
     const Y* y_part = y + token * width + at;
     const T* z_part = z + token * z_stride + at;
-    float kept[kKept];
+    float kept[kKept][kVec];
     float squares = 0.0f;
+    auto gated = [&](int c, float (&v)[kVec]) {
+        float g[kVec];
+        load_some<Y, kVec>(y_part + c, v);
+        load_some<T, kVec>(z_part + c, g);
+#pragma unroll
+        for (int j = 0; j < kVec; ++j) v[j] *= g[j] * sigmoid(g[j]);
+    };
 #pragma unroll
     for (int i = 0; i < kKept; ++i) {
-        const int c = threadIdx.x + i * blockDim.x;
-        kept[i] = 0.0f;
+        const int c = threadIdx.x * kVec + i * step;
         if (c < size) {
-            const float g = Num<T>::load(z_part + c);
-            kept[i] = Num<Y>::load(y_part + c) * (g * sigmoid(g));
+            gated(c, kept[i]);
+#pragma unroll
+            for (int j = 0; j < kVec; ++j) squares = fmaf(kept[i][j], kept[i][j], squares);
         }
-        squares = fmaf(kept[i], kept[i], squares);
     }
-    for (int c = threadIdx.x + kKept * blockDim.x; c < size; c += blockDim.x) {  // (parts too large for the registers are read twice)
-        const float g = Num<T>::load(z_part + c);
-        const float v = Num<Y>::load(y_part + c) * (g * sigmoid(g));
-        squares = fmaf(v, v, squares);
+    for (int c = threadIdx.x * kVec + kKept * step; c < size; c += step) {
+        float v[kVec];
+        gated(c, v);
+#pragma unroll
+        for (int j = 0; j < kVec; ++j) squares = fmaf(v[j], v[j], squares);
     }
     const float factor = out_scale / sqrtf(block_sum(squares, scratch) / (float)size + eps);
+    auto store = [&](int c, float (&v)[kVec]) {
+        float w[kVec];
+        load_some<float, kVec>(gain + at + c, w);
+#pragma unroll
+        for (int j = 0; j < kVec; ++j) v[j] *= factor * w[j];
+        T* dst = out + token * out_stride + at + c;
+        if constexpr (kVec == 8) {
+            store8(dst, v);
+        } else {
+#pragma unroll
+            for (int j = 0; j < kVec; ++j) Num<T>::store(dst + j, v[j]);
+        }
+    };
 #pragma unroll
     for (int i = 0; i < kKept; ++i) {
-        const int c = threadIdx.x + i * blockDim.x;
-        if (c < size) Num<T>::store(out + token * out_stride + at + c, kept[i] * factor * gain[at + c]);
+        const int c = threadIdx.x * kVec + i * step;
+        if (c < size) store(c, kept[i]);
     }
-    for (int c = threadIdx.x + kKept * blockDim.x; c < size; c += blockDim.x) {
-        const float g = Num<T>::load(z_part + c);
-        Num<T>::store(out + token * out_stride + at + c, Num<Y>::load(y_part + c) * (g * sigmoid(g)) * factor * gain[at + c]);
+    for (int c = threadIdx.x * kVec + kKept * step; c < size; c += step) {
+        float v[kVec];
+        gated(c, v);
+        store(c, v);
     }
 }
 
@@ -192,13 +225,18 @@ template <typename T, typename Y>
 int gate_part_norm(const void* y, const void* z, int z_stride, const float* gain, float eps, void* out, int out_stride, float out_scale,
                    int tokens, int width, int parts, cudaStream_t stream) {
     const int size = width / parts;
-    const int threads = size <= 512 ? 128 : 256;
-    if (size <= threads * 4)
-        MB_LAUNCH("gate_part_norm", (gate_part_norm_kernel<T, Y, 4>), dim3(tokens, parts), dim3(threads), 0, stream, true, (const Y*)y, (const T*)z,
-                  z_stride, gain, eps, (T*)out, out_stride, out_scale, width, size);
-    else
-        MB_LAUNCH("gate_part_norm", (gate_part_norm_kernel<T, Y, 16>), dim3(tokens, parts), dim3(threads), 0, stream, true, (const Y*)y, (const T*)z,
-                  z_stride, gain, eps, (T*)out, out_stride, out_scale, width, size);
+    const uintptr_t starts = (uintptr_t)y | (uintptr_t)z | (uintptr_t)gain | (uintptr_t)out;
+    const bool eight = size % 8 == 0 && width % 8 == 0 && !(starts & 15) && ((size_t)z_stride * sizeof(T)) % 16 == 0 && ((size_t)out_stride * sizeof(T)) % 16 == 0;
+    const int vec = eight ? 8 : 1;
+    int threads = 32;
+    while (threads < 256 && threads * vec < size) threads *= 2;
+#define MB_PART(VEC, KEPT)                                                                                                               \
+    MB_LAUNCH("gate_part_norm", (gate_part_norm_kernel<T, Y, VEC, KEPT>), dim3(tokens, parts), dim3(threads), 0, stream, true, (const Y*)y, \
+              (const T*)z, z_stride, gain, eps, (T*)out, out_stride, out_scale, width, size)
+    if (eight && size <= threads * 8) MB_PART(8, 1);
+    else if (eight) MB_PART(8, 4);
+    else MB_PART(1, 8);
+#undef MB_PART
     return 0;
 }
 

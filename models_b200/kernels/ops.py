@@ -1606,6 +1606,44 @@ def skinny_gemm_gated_residual(weight: torch.Tensor, x: torch.Tensor, out: torch
                                                 _p(gate), gate.stride(0), _p(bias), _sm_count(weight.device), 1, _stream()))
 
 
+def skinny_gemm_tanh_residual(weight: torch.Tensor, x: torch.Tensor, out: torch.Tensor, alpha: float, norm_weight: torch.Tensor,
+                              norm_bias: torch.Tensor, then=None) -> Optional[torch.Tensor]:
+    """out += tanh(alpha * (x . weight^T)) * norm_weight + norm_bias for few rows, in the decode product's epilogue.  x bfloat16 [rows, k],
+    weight bfloat16 [n, k], out the contiguous float32 stream [rows, n]; `then` as for result_tanh_add (rows in bfloat16)."""
+    _cuda(weight, x, out, norm_weight, norm_bias)
+    n, k = weight.shape
+    batch = x.shape[0]
+    if x.dtype != torch.bfloat16 or x.stride(1) != 1 or x.shape[1] != k or not skinny_takes(weight, batch):
+        raise KernelError(f"skinny_gemm_tanh_residual does not take a {tuple(weight.shape)} weight with {tuple(x.shape)} {x.dtype} rows")
+    _stream_rows(out, "skinny_gemm_tanh_residual")
+    if tuple(out.shape) != (batch, n):
+        raise KernelError(f"skinny_gemm_tanh_residual: the stream is {tuple(out.shape)}, the product [{batch}, {n}]")
+    _vectors(n, "skinny_gemm_tanh_residual", weight=norm_weight, bias=norm_bias)
+    (kind, then_alpha, then_weight, then_bias, rows_at, _), rows = _then_args(out, then, torch.bfloat16, "skinny_gemm_tanh_residual")
+    lib = skinny()
+    _run(lib, lib.mb_skinny_gemm_tanh_residual(_p(weight), weight.stride(0), n, k, batch, _p(x), x.stride(0), _p(out), out.stride(0),
+                                               ctypes.c_float(alpha), _p(norm_weight), _p(norm_bias), kind, then_alpha, then_weight, then_bias,
+                                               rows_at, n, _sm_count(weight.device), 1, _stream()))
+    return rows
+
+
+def skinny_gemm_side(weight: torch.Tensor, x: torch.Tensor, table: torch.Tensor, tokens: torch.Tensor, columns: int) -> torch.Tensor:
+    """What side_gate makes of the product x . weight^T, in the decode product's epilogue: bfloat16 [rows, columns], weight [columns, k]."""
+    _cuda(weight, x, table, tokens)
+    _int32(tokens, "tokens")
+    n, k = weight.shape
+    batch = x.shape[0]
+    if x.dtype != torch.bfloat16 or x.stride(1) != 1 or x.shape[1] != k or not skinny_takes(weight, batch) or n != columns:
+        raise KernelError(f"skinny_gemm_side does not take a {tuple(weight.shape)} weight with {tuple(x.shape)} {x.dtype} rows")
+    if table.dtype != torch.bfloat16 or table.dim() != 2 or not table.is_contiguous() or table.shape[1] > n or tokens.numel() != batch:
+        raise KernelError(f"skinny_gemm_side: the table {tuple(table.shape)} {table.dtype} does not fit {n} columns")
+    out = torch.empty((batch, n), dtype=torch.bfloat16, device=weight.device)
+    lib = skinny()
+    _run(lib, lib.mb_skinny_gemm_side(_p(weight), weight.stride(0), n, k, batch, _p(x), x.stride(0), _p(out), n, _p(table), _p(tokens),
+                                      table.shape[1], _sm_count(weight.device), 1, _stream()))
+    return out
+
+
 def skinny_qkv_rope(weight: torch.Tensor, xf: Optional[torch.Tensor], gain: Optional[torch.Tensor], eps: float, heads: int,
                     kv_heads: int, head_dim: int, positions: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor,
                     k_pool: torch.Tensor, v_pool: torch.Tensor, slot_mapping: torch.Tensor, x: Optional[torch.Tensor] = None,
@@ -2227,43 +2265,53 @@ GROUPED_ROWS_PER_EXPERT = 32  # from so many entries per expert on average a ste
 EXPERT_ROWS_ENTRIES = 64  # up to so many (token, choice) entries a step's experts run entry by entry, without sorting
 
 
+def _row_choices(chosen: torch.Tensor, tokens: Optional[torch.Tensor], rows: Optional[int], name: str) -> int:
+    """The number of entries: those of `chosen` [rows, top], or with `tokens` (int32 [rows]) of the rows of the table `chosen`
+    [vocab, top] that the ids name."""
+    _cuda(chosen, tokens)
+    _int32(chosen, "chosen")
+    _int32(tokens, "tokens")
+    if chosen.dim() != 2 or not chosen.is_contiguous() or (rows is not None and (chosen if tokens is None else tokens).shape[0] != rows):
+        raise KernelError(f"{name}: choices {tuple(chosen.shape)} do not fit {rows} rows")
+    return chosen.numel() if tokens is None else tokens.numel() * chosen.shape[1]
+
+
 def expert_rows_first(x: torch.Tensor, gate_w: torch.Tensor, up_w: torch.Tensor, chosen: torch.Tensor, limit: float,
-                      slope: float, up_offset: float = 1.0) -> torch.Tensor:
+                      slope: float, up_offset: float = 1.0, tokens: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The first product for a step of few tokens: mid [tokens * top, n] (row token * top + choice, x's dtype), each row
     clamped_swish(gate_w[e] . x, up_w[e] . x) for its token's row x and its chosen expert e.  Every entry streams its
-    expert's matrices once; nothing is sorted."""
+    expert's matrices once; nothing is sorted.  With `tokens` (int32 [tokens]) `chosen` is a table [vocab, top] read by token id."""
     _cuda(x, gate_w, up_w, chosen)
     _columns(x, "x")
-    _int32(chosen, "chosen")
+    entries = _row_choices(chosen, tokens, x.shape[0], "expert_rows_first")
     experts = gate_w.shape[0]
     _expert_weights(gate_w, experts, "expert_rows_first")
     _expert_weights(up_w, experts, "expert_rows_first")
-    if gate_w.shape != up_w.shape or gate_w.shape[2] != x.shape[1] or not (gate_w.dtype == up_w.dtype == x.dtype) \
-            or chosen.dim() != 2 or chosen.shape[0] != x.shape[0] or not chosen.is_contiguous():
+    if gate_w.shape != up_w.shape or gate_w.shape[2] != x.shape[1] or not (gate_w.dtype == up_w.dtype == x.dtype):
         raise KernelError(f"expert_rows_first: matrices {tuple(gate_w.shape)} / {tuple(up_w.shape)} and choices {tuple(chosen.shape)} "
                           f"do not fit rows {tuple(x.shape)}")
     n, k, top = gate_w.shape[1], gate_w.shape[2], chosen.shape[1]
-    mid = torch.empty((chosen.numel(), n), dtype=x.dtype, device=x.device)
+    mid = torch.empty((entries, n), dtype=x.dtype, device=x.device)
     lib = routed_experts_library()
-    _run(lib, lib.mb_expert_rows(_p(x), x.stride(0), _p(gate_w), _p(up_w), _p(mid), None, n, _code(x.dtype), _p(chosen), chosen.numel(),
+    _run(lib, lib.mb_expert_rows(_p(x), x.stride(0), _p(gate_w), _p(up_w), _p(mid), None, n, _code(x.dtype), _p(chosen), _p(tokens), entries,
                                  top, experts, n, k, ctypes.c_float(limit), ctypes.c_float(slope), ctypes.c_float(up_offset), 1, _stream()))
     return mid
 
 
-def expert_rows_second(mid: torch.Tensor, down_w: torch.Tensor, chosen: torch.Tensor) -> torch.Tensor:
+def expert_rows_second(mid: torch.Tensor, down_w: torch.Tensor, chosen: torch.Tensor, tokens: Optional[torch.Tensor] = None) -> torch.Tensor:
     """slot_out float32 [tokens * top, n]: row i is down_w[e_i] . mid[i] for entry i's chosen expert (float32 sums)."""
     _cuda(mid, down_w, chosen)
-    _int32(chosen, "chosen")
+    entries = _row_choices(chosen, tokens, None, "expert_rows_second")
     experts = down_w.shape[0]
     _expert_weights(down_w, experts, "expert_rows_second")
-    if mid.dim() != 2 or not mid.is_contiguous() or mid.shape[0] != chosen.numel() or down_w.shape[2] != mid.shape[1] \
-            or down_w.dtype != mid.dtype or not chosen.is_contiguous():
+    if mid.dim() != 2 or not mid.is_contiguous() or mid.shape[0] != entries or down_w.shape[2] != mid.shape[1] \
+            or down_w.dtype != mid.dtype:
         raise KernelError(f"expert_rows_second: matrices {tuple(down_w.shape)} do not fit rows {tuple(mid.shape)}")
     n, k = down_w.shape[1], down_w.shape[2]
     slot_out = torch.empty((mid.shape[0], n), dtype=torch.float32, device=mid.device)
     lib = routed_experts_library()
     _run(lib, lib.mb_expert_rows(_p(mid), mid.stride(0), _p(down_w), None, None, _p(slot_out), n, _code(mid.dtype), _p(chosen),
-                                 chosen.numel(), chosen.shape[1], experts, n, k, ctypes.c_float(0.0), ctypes.c_float(0.0), ctypes.c_float(0.0), 0, _stream()))
+                                 _p(tokens), entries, chosen.shape[1], experts, n, k, ctypes.c_float(0.0), ctypes.c_float(0.0), ctypes.c_float(0.0), 0, _stream()))
     return slot_out
 
 

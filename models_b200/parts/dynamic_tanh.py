@@ -49,5 +49,13 @@ class DynamicTanh(Part):
             y = y.rows
         return ops.result_tanh_add(x, y, self.alpha, self.weight, self.bias, then, self.runtime.compute_dtype, **entries)
 
+    def add_product(self, x: torch.Tensor, a: torch.Tensor, weight: torch.Tensor, then):
+        """x += norm(a . weight^T), or None if the product's kernel has no such epilogue (many rows, other types or sizes): with few
+        rows (decode) norm, addition and the next reader's rows ride in the product.  Returns (rows of `then`,)."""
+        if (self.runtime.mode == "bfloat16" and weight.dtype == torch.bfloat16 and a.dtype == torch.bfloat16 and ops.skinny_pays(weight, a.shape[0])
+                and a.stride(0) % 8 == 0 and a.data_ptr() % 16 == 0):
+            return (ops.skinny_gemm_tanh_residual(weight, a, x, self.alpha, self.weight, self.bias, then),)
+        return None
+
 
 register_part("norm", "dynamic_tanh", DynamicTanh)

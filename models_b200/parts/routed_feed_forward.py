@@ -115,18 +115,22 @@ class RoutedFeedForward(Part):
             self.shared_in, self.shared_starts = stack_rows(first)
             self.shared_down = rt.matrix(tensors[n["shared_down"]])
 
-    def _experts(self, x: torch.Tensor, chosen: torch.Tensor):
-        """The chosen experts' float32 results and the row of every (token, choice) entry among them (None: in entry order)."""
+    def _experts(self, x: torch.Tensor, chosen: Optional[torch.Tensor], tokens: Optional[torch.Tensor] = None):
+        """The chosen experts' float32 results and the row of every (token, choice) entry among them (None: in entry order).
+        `tokens`: the choices are the table's rows of these ids (`chosen` None)."""
         s = self.spec
         e = s.expert
         position = None
         # (an identity expert's id lies beyond the experts': the sorting and the products leave its entries out, and the
         # weighted sum takes the token's own row for them)
-        if chosen.numel() <= ops.EXPERT_ROWS_ENTRIES:
+        if x.shape[0] * s.top <= ops.EXPERT_ROWS_ENTRIES:
             # a decode step: every entry streams its expert's matrices; no sorting, no tiles of mostly empty rows
-            mid = ops.expert_rows_first(x, self.w_gate, self.w_up, chosen, e.limit, e.swish_slope, e.up_offset)
-            slot_out = ops.expert_rows_second(mid, self.w_down, chosen)
-        elif self.grouped and chosen.numel() >= ops.GROUPED_ROWS_PER_EXPERT * s.num_experts:
+            ids = chosen if tokens is None else self.table
+            mid = ops.expert_rows_first(x, self.w_gate, self.w_up, ids, e.limit, e.swish_slope, e.up_offset, tokens)
+            return ops.expert_rows_second(mid, self.w_down, ids, tokens), None
+        if tokens is not None:
+            chosen = ops.table_route(self.table, tokens)
+        if self.grouped and chosen.numel() >= ops.GROUPED_ROWS_PER_EXPERT * s.num_experts:
             # a prompt: every expert's rows fill tiles of their own, and both products run on the tcgen05 tensor cores
             plan = ops.route_pad(chosen, s.num_experts)
             mid = ops.grouped_first_product(ops.gather_rows(x, plan), self.w_gate_up, plan, e.limit, e.swish_slope, e.up_offset)
@@ -139,7 +143,7 @@ class RoutedFeedForward(Part):
 
     def _forward_results(self, xn: torch.Tensor, batch, run=None) -> ExpertResults:
         x = xn if xn.dtype == self.w_down.dtype else xn.to(self.w_down.dtype)
-        rows, position = self._experts(x, ops.table_route(self.table, batch.tokens))
+        rows, position = self._experts(x, None, batch.tokens)
         return ExpertResults(rows, position, self.spec.top, 1.0 / self.spec.top)
 
     def forward_wide(self, xn: torch.Tensor, batch=None, run=None) -> torch.Tensor:

@@ -8,7 +8,8 @@ The norms before a sublayer are dynamic tanhs: they need no sum over a row, so t
 float32 stream also makes the next reader's rows -- the feed-forward's, the side input's (the stream itself in the compute type),
 and, handed on as StreamRows, the next layer's.  The norms on the results offer `add_result` (a dynamic tanh, an RMS norm).
 A sublayer is a part with `forward_results` (expert results still to be summed), with `forward_wide` (float32 rows), or a split
-part (a first product, something in between, a last product whose float32 sums are the result).
+part (a first product, something in between, a last product whose float32 sums are the result; with few rows the norm on
+the result and the addition ride in that product's epilogue where the norm offers it, `add_product`).
 """
 
 from __future__ import annotations
@@ -53,17 +54,19 @@ class SandwichBlock(Part):
         for part in self.parts:
             part.load(tensors)
 
-    def _result(self, part, rows, batch, run):
+    def _sublayer(self, x, part, after, rows, batch, run, then):
+        """x += after(part(rows)); returns the rows that `then` asks for."""
         if hasattr(part, "forward_results"):
-            return part.forward_results(rows, batch, run)
+            return after.add_result(x, part.forward_results(rows, batch, run), then)
         if hasattr(part, "forward_wide"):
-            return part.forward_wide(rows, batch, run)
+            return after.add_result(x, part.forward_wide(rows, batch, run), then)
         dtype = self.runtime.compute_dtype
         w_in, w_out = part.input_matrix(), part.output_matrix()
         proj = linear(rows, w_in, dtype)
         mid = torch.empty((rows.shape[0], w_out.shape[1]), dtype=dtype, device=rows.device)
         part.inner(proj[:, :w_in.shape[0]], mid, batch, run, 1.0)
-        return linear(mid, w_out, torch.float32)
+        done = after.add_product(x, mid, w_out, then) if hasattr(after, "add_product") else None
+        return done[0] if done is not None else after.add_result(x, linear(mid, w_out, torch.float32), then)
 
     def forward(self, x: torch.Tensor, pending, batch, run: RunContext, following=None):
         """`pending`: None, a delta still to be added, or the rows the block before left for this one (a StreamRows).
@@ -84,8 +87,7 @@ class SandwichBlock(Part):
                 then = before.then_args() if before is not None else (None if float_mode else "rows")
             else:
                 then = following.mixer_norm.then_args() if hand_on else None
-            result = self._result(part, rows, batch, run)
-            rows = after.add_result(x, result, then)
+            rows = self._sublayer(x, part, after, rows, batch, run, then)
             if rows is None:
                 rows = x
         return StreamRows(rows, following) if hand_on else None

@@ -30,8 +30,12 @@ class TokenSide(Part):
 
     def forward_wide(self, xn: torch.Tensor, batch, run=None) -> torch.Tensor:
         """xn: the stream's rows in the compute type; float32 [tokens, width]."""
-        gate = linear(xn, self.gate, torch.float32)
-        return linear(ops.side_gate(gate, self.table, batch.tokens, self.proj.shape[1]), self.proj, torch.float32)
+        if (xn.dtype == torch.bfloat16 and self.gate.dtype == torch.bfloat16 and ops.skinny_pays(self.gate, xn.shape[0])
+                and xn.stride(0) % 8 == 0 and xn.data_ptr() % 16 == 0):
+            gated = ops.skinny_gemm_side(self.gate, xn, self.table, batch.tokens, self.proj.shape[1])  # few rows: in the product's epilogue
+        else:
+            gated = ops.side_gate(linear(xn, self.gate, torch.float32), self.table, batch.tokens, self.proj.shape[1])
+        return linear(gated, self.proj, torch.float32)
 
 
 register_part("feed_forward", "token_side", TokenSide)
