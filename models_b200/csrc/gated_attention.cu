@@ -832,6 +832,82 @@ __global__ void head_linear_kernel(const T* __restrict__ in, int in_stride, cons
     }
 }
 
+// The same product for a decode step's few tokens (up to 8, bfloat16, n_in a multiple of 8 up to 256 * kChunks, rows on 16 bytes): grid
+// (ceil(n_out / (4 warps * kPasses * rows per pass)), heads); block 128.  kLanes lanes share a weight row in 16-byte pieces, a warp takes
+// 32 / kLanes rows per pass; all of a warp's weights are asked for before the wait for the kernel that makes the tokens' rows.
+template <int kLanes, int kPasses, int kChunks>
+__global__ void __launch_bounds__(128)
+head_linear_few_kernel(const __nv_bfloat16* __restrict__ in, int in_stride, const __nv_bfloat16* __restrict__ w, __nv_bfloat16* __restrict__ out,
+                       int out_stride, const __nv_bfloat16* __restrict__ gate, int gate_stride, int tokens, int n_in, int n_out, HeadLayout layout) {
+    using bf16 = __nv_bfloat16;
+    grid_launch_dependents();
+    constexpr int kRowsPerPass = 32 / kLanes, kTokens = 8;
+    const int head = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, part = lane % kLanes, sub_row = lane / kLanes;
+    const int row0 = (blockIdx.x * 4 + warp) * kPasses * kRowsPerPass;
+    uint4 weight[kPasses][kChunks];
+#pragma unroll
+    for (int p = 0; p < kPasses; ++p)
+#pragma unroll
+        for (int c = 0; c < kChunks; ++c) {
+            const int n = row0 + p * kRowsPerPass + sub_row, k = (c * kLanes + part) * 8;
+            weight[p][c] = make_uint4(0u, 0u, 0u, 0u);
+            if (n < n_out && k < n_in) weight[p][c] = *reinterpret_cast<const uint4*>(w + ((size_t)head * n_out + n) * n_in + k);
+        }
+    grid_dependency_wait();
+    if (layout.turned > 0 && blockIdx.x == 0) {
+        const int half = layout.turned / 2;
+        for (int item = threadIdx.x; item < tokens * half; item += blockDim.x) {
+            const size_t row = item / half;
+            turn_tail<bf16>(in + row * in_stride + (size_t)head * layout.in_head + n_in, out + row * out_stride + (size_t)head * layout.out_head + n_out,
+                            item % half, layout, layout.positions[row]);
+        }
+    }
+    float acc[kPasses][kTokens];
+#pragma unroll
+    for (int p = 0; p < kPasses; ++p)
+#pragma unroll
+        for (int t = 0; t < kTokens; ++t) acc[p][t] = 0.0f;
+#pragma unroll
+    for (int c = 0; c < kChunks; ++c) {
+        const int k = (c * kLanes + part) * 8;
+        uint4 raw[kTokens];
+#pragma unroll
+        for (int t = 0; t < kTokens; ++t) {
+            raw[t] = make_uint4(0u, 0u, 0u, 0u);
+            if (t < tokens && k < n_in) raw[t] = *reinterpret_cast<const uint4*>(in + (size_t)t * in_stride + (size_t)head * layout.in_head + k);
+        }
+#pragma unroll
+        for (int t = 0; t < kTokens; ++t) {
+            const uint32_t x[4] = {raw[t].x, raw[t].y, raw[t].z, raw[t].w};
+#pragma unroll
+            for (int p = 0; p < kPasses; ++p) {
+                const uint32_t v[4] = {weight[p][c].x, weight[p][c].y, weight[p][c].z, weight[p][c].w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    acc[p][t] = fmaf(__uint_as_float(x[i] << 16), __uint_as_float(v[i] << 16), acc[p][t]);
+                    acc[p][t] = fmaf(__uint_as_float(x[i] & 0xffff0000u), __uint_as_float(v[i] & 0xffff0000u), acc[p][t]);
+                }
+            }
+        }
+    }
+#pragma unroll
+    for (int p = 0; p < kPasses; ++p) {
+        const int n = row0 + p * kRowsPerPass + sub_row;
+        float mine = 0.0f;
+#pragma unroll
+        for (int t = 0; t < kTokens; ++t) {
+            float total = acc[p][t];
+#pragma unroll
+            for (int offset = 1; offset < kLanes; offset <<= 1) total += __shfl_xor_sync(0xffffffffu, total, offset);
+            if (part == t) mine = total;  // lane `part` of the row's lanes stores token `part`'s result
+        }
+        if (part < tokens && part < kTokens && n < n_out) {
+            if (gate != nullptr) mine *= sigmoid(__bfloat162float(gate[(size_t)part * gate_stride + (layout.element_gate ? head * n_out + n : head)]));
+            out[(size_t)part * out_stride + (size_t)head * layout.out_head + n] = __float2bfloat16_rn(mine);
+        }
+    }
+}
+
 // The same product on the tensor cores, for bfloat16 steps of many tokens: grid (ceil(tokens / 64), heads); block 128,
 // a warp 16 tokens.  The head's 64 x n_in activations and, 64 rows at a time, its weights pass through shared memory
 // (cp.async, two stages); m16n8k16 products with float sums.  n_in and n_out are multiples of 16.
@@ -1228,6 +1304,22 @@ MB_EXPORT int mb_head_linear(const void* in, int in_stride, const void* w, void*
                   gate_stride, tokens, n_in, n_out, layout);
         return check_launch("head_linear_tc");
     }
+    if (tensor_cores && dtype == MB_BF16 && tokens <= 8 && n_in % 8 == 0 && n_in <= 512 && in_stride % 8 == 0 && in_head % 8 == 0 && !((uintptr_t)in & 15) &&
+        !((uintptr_t)w & 15)) {
+#define MB_FEW(LANES, PASSES, CHUNKS)                                                                                                     \
+    do {                                                                                                                                  \
+        constexpr int kBlockRows = 4 * (PASSES) * (32 / (LANES));                                                                          \
+        MB_LAUNCH("head_linear_few", (head_linear_few_kernel<LANES, PASSES, CHUNKS>), dim3((n_out + kBlockRows - 1) / kBlockRows, heads), dim3(128), 0, \
+                  stream, true, (const __nv_bfloat16*)in, in_stride, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, out_stride,             \
+                  (const __nv_bfloat16*)gate, gate_stride, tokens, n_in, n_out, layout);                                                   \
+        return check_launch("head_linear_few");                                                                                           \
+    } while (0)
+        if (n_in <= 64) MB_FEW(8, 2, 1);
+        if (n_in <= 128) MB_FEW(16, 4, 1);
+        if (n_in <= 256) MB_FEW(32, 4, 1);
+        MB_FEW(32, 4, 2);
+#undef MB_FEW
+    }
     const size_t smem = (size_t)kHeadRows * n_in * sizeof(float);
     if (smem > 200 * 1024) return fail("head_linear: %d inputs per head exceed a block's shared memory", n_in);
     const dim3 grid((tokens + kHeadRows - 1) / kHeadRows, heads, (n_out + kHeadOutputs - 1) / kHeadOutputs);
@@ -1294,4 +1386,18 @@ MB_EXPORT int mb_latent_prepare(const void* q, int q_stride, const float* q_gain
     else
         return fail("latent_prepare: unknown dtype code %d", dtype);
     return check_launch("latent_prepare");
+}
+
+// The second half of mb_gated_attention_decode alone: adds the runs that another kernel left in `partial` (bfloat16 results, softmax).
+MB_EXPORT int mb_gated_attention_combine(const float* partial, int splits, void* out, int out_stride, const int* cu_q, const int* kv_lens,
+                                         const void* gate, int gate_stride, int gate_kind, int sequences, int heads, int value_dim, int sink,
+                                         cudaStream_t stream) {
+    if (sequences <= 0) return 0;
+    if (value_dim <= 0 || value_dim > 512 || gate_kind < 0 || gate_kind > 2 || (gate_kind != 0 && gate == nullptr))
+        return fail("gated_attention_combine: value_dim %d, gate kind %d", value_dim, gate_kind);
+    const ScoreExtras extras{nullptr, 0.0f, sink, nullptr, nullptr, 0, 0};
+    MB_LAUNCH("gated_attention_combine", (gated_attention_combine_kernel<__nv_bfloat16, true>), dim3(heads, sequences), dim3((value_dim + 31) / 32 * 32), 0,
+              stream, true, partial, splits, (__nv_bfloat16*)out, out_stride, cu_q, (const __nv_bfloat16*)gate, gate_stride, gate_kind, heads,
+              value_dim, kv_lens, extras);
+    return check_launch("gated_attention_combine");
 }

@@ -353,9 +353,218 @@ gated_attention_tc_kernel(const bf16* __restrict__ q, int q_stride, bf16* __rest
 
 constexpr size_t kSmemBytes = (size_t)kQRows * kKeyRow + 2 * (size_t)kStageBytes;
 
+#if MB_SHARED_ROWS
+// ------------------------------------------------------------------------------------------------
+// Decoding over rows that all heads share (one query token per sequence, softmax weights): sixteen heads' queries are one 16-row
+// operand, so a page of rows is read once for all of them.  grid (runs, head tiles of 16, sequences); block 128.  A run is `span` pages,
+// counted from the first page the query sees; pages arrive through two stages of cp.async copies.  Of a page, warp w takes the keys
+// 16 w .. 16 w + 15 for the scores; the warps meet for the rows' maxima and put the weights, each as two bfloat16 numbers, in shared
+// memory; then warp w takes the value columns of the 16-column tiles w, w + 4, ...  Every run leaves [maximum, sum of weights, VD sums]
+// per head for the kernel that adds the runs up; a run behind the sequence's end leaves a sum of 0.
+constexpr int kWeightRow = kTile * 2 + 16;
+constexpr int kValueTiles = (VD / 16 + 3) / 4;  // of a warp
+constexpr size_t kDecodeBytes = 16 * (size_t)kKeyRow + 2 * (size_t)kKeyTile + 2 * 16 * (size_t)kWeightRow;
+
+__global__ void __launch_bounds__(kThreads)
+gated_attention_tc_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restrict__ k_pool, const int* __restrict__ block_table,
+                                 int max_blocks, const int* __restrict__ cu_q, const int* __restrict__ kv_lens, float* __restrict__ partial,
+                                 int span, int heads, float scale, ScoreExtras extras) {
+    grid_launch_dependents();
+    grid_dependency_wait();
+    extern __shared__ __align__(16) unsigned char smem[];
+    __shared__ float warp_max_s[4][16], warp_sum_s[4][16];
+    unsigned char* q_smem = smem;
+    unsigned char* stage_smem = smem + 16 * kKeyRow;
+    unsigned char* weight_smem = stage_smem + 2 * kKeyTile;  // [hi, lo][16][64]
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, group_id = lane >> 2, tid4 = lane & 3;
+    const int seq = blockIdx.z, run = blockIdx.x, runs = gridDim.x, head0 = blockIdx.y * 16;
+    const int count = min(16, heads - head0);
+    const int pos = kv_lens[seq] - 1;
+    const int lowest = lowest_visible(pos, extras);
+    const int first_page = lowest / kTile + run * span, end_page = min(pos / kTile + 1, first_page + span);
+    constexpr int kStride = 2 + VD;
+    float* mine = partial + (((size_t)seq * heads + head0) * runs + run) * kStride;  // the head's rows lie runs * kStride apart
+    if (first_page >= end_page) {
+        for (int h = threadIdx.x; h < count; h += kThreads) {
+            mine[(size_t)h * runs * kStride] = -CUDART_INF_F;
+            mine[(size_t)h * runs * kStride + 1] = 0.0f;
+        }
+        return;
+    }
+    const int* table = block_table + (size_t)seq * max_blocks;
+    const uint32_t stage_base = smem_u32(stage_smem);
+    load_tile<KD, kKeyRow>(stage_base, k_pool, table[first_page], 0, 1);
+    cp_async_commit();
+    {
+        constexpr int kPieces = KD / 8;
+        const bf16* first = q + (size_t)cu_q[seq] * q_stride + (size_t)head0 * KD;
+        for (int i = threadIdx.x; i < 16 * kPieces; i += kThreads) {
+            const int row = i / kPieces, piece = i % kPieces;
+            uint4 v = make_uint4(0u, 0u, 0u, 0u);
+            if (row < count) v = *reinterpret_cast<const uint4*>(first + (size_t)row * KD + piece * 8);
+            *reinterpret_cast<uint4*>(q_smem + row * kKeyRow + piece * 16) = v;
+        }
+    }
+    constexpr float kLog2e = 1.4426950408889634f;
+    const uint32_t q_rows = smem_u32(q_smem) + ((lane & 7) + ((lane >> 3) & 1) * 8) * kKeyRow + (lane >> 4) * 16;
+    const uint32_t weight_rows = smem_u32(weight_smem) + ((lane & 7) + ((lane >> 3) & 1) * 8) * kWeightRow + (lane >> 4) * 16;
+    float o[kValueTiles][2][4];
+#pragma unroll
+    for (int i = 0; i < kValueTiles; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) o[i][0][j] = o[i][1][j] = 0.0f;
+    float run_max[2] = {-CUDART_INF_F, -CUDART_INF_F}, run_sum[2] = {0.0f, 0.0f};  // of rows group_id and group_id + 8
+    for (int page = first_page; page < end_page; ++page) {
+        const int stage = (page - first_page) & 1;
+        if (page + 1 < end_page) {
+            load_tile<KD, kKeyRow>(stage_base + (stage ^ 1) * kKeyTile, k_pool, table[page + 1], 0, 1);
+            cp_async_commit();
+            cp_async_wait<1>();
+        } else {
+            cp_async_wait<0>();
+        }
+        __syncthreads();
+        const uint32_t tile = stage_base + stage * kKeyTile;
+        const int key_base = page * kTile;
+        const int stale_from = pos + 1 - key_base, unseen = lowest - key_base;
+        if (stale_from < kTile || unseen > 0) {  // rows nobody sees are cleared: a weight of 0 times a stray NaN is NaN
+            unsigned char* rows = stage_smem + stage * kKeyTile;
+            constexpr int kPieces = kKeyRow / 16;
+            for (int i = threadIdx.x; i < kTile * kPieces; i += kThreads) {
+                const int row = i / kPieces;
+                if (row >= stale_from || row < unseen) *reinterpret_cast<uint4*>(rows + row * kKeyRow + (i % kPieces) * 16) = make_uint4(0u, 0u, 0u, 0u);
+            }
+            __syncthreads();
+        }
+        float s[2][4] = {{0.0f, 0.0f, 0.0f, 0.0f}, {0.0f, 0.0f, 0.0f, 0.0f}};
+        const uint32_t key = tile + (warp * 16 + (lane & 7) + ((lane >> 4) & 1) * 8) * kKeyRow + ((lane >> 3) & 1) * 16;
+#pragma unroll 4
+        for (int ks = 0; ks < kKSteps; ++ks) {
+            uint32_t a[4], b[4];
+            ldmatrix_x4(a, q_rows + ks * 32);
+            ldmatrix_x4(b, key + ks * 32);
+            mma_bf16(s[0], a, b[0], b[1]);
+            mma_bf16(s[1], a, b[2], b[3]);
+        }
+        float part_max[2] = {-CUDART_INF_F, -CUDART_INF_F};
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int p = key_base + warp * 16 + nt * 8 + tid4 * 2 + (i & 1);
+                s[nt][i] = p <= pos && p >= lowest ? s[nt][i] * scale : -CUDART_INF_F;
+                part_max[i >> 1] = fmaxf(part_max[i >> 1], s[nt][i]);
+            }
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            const float m = quad_max(part_max[r]);
+            if (tid4 == 0) warp_max_s[warp][group_id + 8 * r] = m;
+        }
+        __syncthreads();
+        float correction[2];
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            const int row = group_id + 8 * r;
+            const float page_max = fmaxf(fmaxf(warp_max_s[0][row], warp_max_s[1][row]), fmaxf(warp_max_s[2][row], warp_max_s[3][row]));
+            const float new_max = fmaxf(run_max[r], page_max);  // finite: every page of the run holds a visible key
+            correction[r] = fast_exp2((run_max[r] - new_max) * kLog2e);
+            run_max[r] = new_max;
+            run_sum[r] *= correction[r];
+        }
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+            for (int r = 0; r < 2; ++r) {
+                const float e0 = fast_exp2((s[nt][2 * r] - run_max[r]) * kLog2e), e1 = fast_exp2((s[nt][2 * r + 1] - run_max[r]) * kLog2e);
+                run_sum[r] += e0 + e1;  // (this lane's keys only; the lanes and warps are added up at the end)
+                uint32_t hi, lo;
+                split_pair(e0, e1, hi, lo);
+                unsigned char* dst = weight_smem + (group_id + 8 * r) * kWeightRow + (warp * 16 + nt * 8 + tid4 * 2) * 2;
+                *reinterpret_cast<uint32_t*>(dst) = hi;
+                *reinterpret_cast<uint32_t*>(dst + 16 * kWeightRow) = lo;
+            }
+#pragma unroll
+        for (int i = 0; i < kValueTiles; ++i)
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                o[i][half][0] *= correction[0], o[i][half][1] *= correction[0];
+                o[i][half][2] *= correction[1], o[i][half][3] *= correction[1];
+            }
+        __syncthreads();
+#pragma unroll
+        for (int part = 0; part < kTile / 16; ++part) {
+            uint32_t hi[4], lo[4];
+            ldmatrix_x4(hi, weight_rows + part * 32);
+            ldmatrix_x4(lo, weight_rows + 16 * kWeightRow + part * 32);
+            const uint32_t value = tile + (part * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kKeyRow + (lane >> 4) * 16;
+#pragma unroll
+            for (int i = 0; i < kValueTiles; ++i) {
+                const int dp = warp + 4 * i;
+                if (dp * 16 >= VD) continue;
+                uint32_t b[4];
+                ldmatrix_x4_trans(b, value + dp * 32);
+                mma_bf16(o[i][0], hi, b[0], b[1]);
+                mma_bf16(o[i][1], hi, b[2], b[3]);
+                mma_bf16(o[i][0], lo, b[0], b[1]);
+                mma_bf16(o[i][1], lo, b[2], b[3]);
+            }
+        }
+        __syncthreads();  // the page's stage and the weights may be written again
+    }
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+        const float total = quad_sum(run_sum[r]);
+        if (tid4 == 0) warp_sum_s[warp][group_id + 8 * r] = total;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+        const int row = group_id + 8 * r;
+        if (row >= count) continue;
+        float* dst = mine + (size_t)row * runs * kStride;
+        if (warp == 0 && tid4 == 0) {
+            dst[0] = run_max[r];
+            dst[1] = warp_sum_s[0][row] + warp_sum_s[1][row] + warp_sum_s[2][row] + warp_sum_s[3][row];
+        }
+#pragma unroll
+        for (int i = 0; i < kValueTiles; ++i) {
+            const int dp = warp + 4 * i;
+            if (dp * 16 >= VD) continue;
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {  // (a head's partial row starts on 8 bytes: 2 + VD is even)
+                *reinterpret_cast<float2*>(dst + 2 + dp * 16 + half * 8 + tid4 * 2) = make_float2(o[i][half][2 * r], o[i][half][2 * r + 1]);
+            }
+        }
+    }
+}
+#endif
+
 }  // namespace mb
 
 using namespace mb;
+
+#if MB_SHARED_ROWS
+// The runs of a decode step over shared rows (one kv head, softmax): `partial` as in csrc/gated_attention.cu, whose combining kernel
+// follows.  q rows of `heads` heads of KD (stride a multiple of 8, 16-byte aligned).
+MB_EXPORT int mb_gated_attention_tc_decode(const void* q, int q_stride, const void* k_pool, const int* block_table, int max_blocks, const int* cu_q,
+                                           const int* kv_lens, float* partial, int runs, int span, int sequences, int heads, int page_size,
+                                           float scale, int block, int window, cudaStream_t stream) {
+    if (sequences <= 0) return 0;
+    if (page_size != kTile || runs < 1 || span < 1) return fail("gated_attention_tc_decode: pages of %d, %d runs of %d pages", page_size, runs, span);
+    if (sequences > 65535 || heads > 65535 * 16) return fail("gated_attention_tc_decode: %d sequences or %d heads exceed the grid limit", sequences, heads);
+    if (q_stride % 8 || ((uintptr_t)q & 15) || ((uintptr_t)k_pool & 15) || ((uintptr_t)partial & 7)) return fail("gated_attention_tc_decode: rows must start on 16 bytes");
+    const ScoreExtras extras{nullptr, 0.0f, 0, nullptr, nullptr, block, window};
+    static bool reserved = false;
+    if (!reserved) {
+        if (cudaFuncSetAttribute(gated_attention_tc_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kDecodeBytes) != cudaSuccess)
+            return fail("gated_attention_tc_decode: cannot reserve %zu bytes of shared memory", kDecodeBytes);
+        reserved = true;
+    }
+    MB_LAUNCH("gated_attention_tc_decode", gated_attention_tc_decode_kernel, dim3(runs, (heads + 15) / 16, sequences), dim3(kThreads), kDecodeBytes,
+              stream, true, (const bf16*)q, q_stride, (const bf16*)k_pool, block_table, max_blocks, cu_q, kv_lens, partial, span, heads, scale, extras);
+    return check_launch("gated_attention_tc_decode");
+}
+#endif
 
 MB_EXPORT int mb_gated_attention_tc_key_dim() { return KD; }
 MB_EXPORT int mb_gated_attention_tc_value_dim() { return VD; }

@@ -835,11 +835,12 @@ def gated_attention(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, v_
     sequence's position 0; `window` n > 0: only if i - j < n.
     `kernel`: None picks the decode form for steps of one token per sequence (the keys cut into runs with a block each;
     the grid follows the page table's width, not the lengths, so that a captured step stays valid), the tensor-core form
-    where it applies (bfloat16 steps of many tokens), else the form with a warp per (token, head); "decode", "tc" or
-    "rows" asks for one of them."""
+    where it applies (bfloat16 steps of many tokens), else the form with a warp per (token, head); decode steps of 8 heads and
+    more over rows they share run on the tensor cores, "tc_decode", where the sizes allow; "decode", "tc", "tc_decode" or "rows"
+    asks for one of them."""
     if weights not in ("softmax", "sigmoid"):
         raise KernelError(f"gated_attention: weights must be 'softmax' or 'sigmoid', got {weights!r}")
-    if kernel not in (None, "tc", "rows", "decode"):
+    if kernel not in (None, "tc", "rows", "decode", "tc_decode"):
         raise KernelError(f"gated_attention: unknown kernel {kernel!r}")
     if gate_kind not in GATE_KINDS or (gate_kind is None) != (gate is None):
         raise KernelError(f"gated_attention: gate kind {gate_kind!r} does not fit the gate given")
@@ -885,6 +886,29 @@ def gated_attention(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, v_
     softmax = 1 if weights == "softmax" else 0
     sequences = kv_lens.numel()
     gate_stride = gate.stride(0) if gate is not None else 0
+    plain_scores = head_scale is None and head_bias is None and softcap == 0.0 and slope_exponent == 0.0 and turn_cos is None
+    shared_decode = (v_pool is None and kv_heads == 1 and heads >= 8 and weights == "softmax" and plain_scores and max_q_len == 1
+                     and gated_attention_tc_takes(q, out, k_pool, head_dim, value_dim, GATED_TC_MIN_ROWS, None))
+    if kernel == "tc_decode" or (kernel is None and shared_decode):
+        # one query token of many heads over rows they all share: sixteen heads are a tensor-core operand
+        if not shared_decode:
+            raise KernelError("the tensor-core decode form takes one bfloat16 token per sequence, 8 heads and more over one head of shared rows, "
+                              "softmax weights of plain scores, and the sizes of the tensor-core form")
+        pages = block_table.shape[1]
+        for seen in (block, window):
+            if seen:
+                pages = min(pages, -(-(seen - 1) // page_size) + 1)
+        span = -(-pages // max(1, min(64, 4 * _sm_count(q.device) // (sequences * -(-heads // 16)))))
+        runs = -(-pages // span)
+        partial = torch.empty((sequences * heads * runs * (2 + value_dim),), dtype=torch.float32, device=q.device)
+        lib = gated_attention_tc_library(head_dim, value_dim, True)
+        _run(lib, lib.mb_gated_attention_tc_decode(_p(q), q.stride(0), _p(k_pool), _p(block_table), block_table.shape[1], _p(cu_q), _p(kv_lens),
+                                                   _p(partial), runs, span, sequences, heads, page_size, ctypes.c_float(scale), int(block),
+                                                   int(window), _stream()))
+        lib = gated_attention_library()
+        _run(lib, lib.mb_gated_attention_combine(_p(partial), runs, _p(out), out.stride(0), _p(cu_q), _p(kv_lens), _p(gate), gate_stride,
+                                                 GATE_KINDS[gate_kind], sequences, heads, value_dim, 1 if sink else 0, _stream()))
+        return
     if kernel == "decode" or (kernel is None and max_q_len == 1):
         if max_q_len != 1:
             raise KernelError("the decode form takes one token per sequence")

@@ -218,7 +218,7 @@ def _plain_attend(q, rows, value_dim, scale, window):
 
 
 FORMS = [("float32", "rows", 64), ("float32", "decode", 64), ("bfloat16", "rows", 64), ("bfloat16", "tc", 64), ("bfloat16", "decode", 64),
-         ("float32", "decode", 32)]
+         ("float32", "decode", 32), ("bfloat16", "tc_decode", 64)]
 
 
 @pytest.mark.parametrize("dtype,kernel,page_size", FORMS)
@@ -230,7 +230,7 @@ def test_one_loud_key_at_the_windows_edge(cuda_device, dtype, kernel, page_size,
     query does not see may hold anything (NaN) when the whole page before the window does."""
     from models_b200.kernels import ops
 
-    H, D, Dv = 3, 48, 32
+    H, D, Dv = 19 if kernel == "tc_decode" else 3, 48, 32
     td = TORCH[dtype]
     g = torch.Generator().manual_seed(T + (window or 0))
     q, rows = torch.randn(T, H, D, generator=g) * 0.3, torch.randn(T, D, generator=g) * 0.3
@@ -239,7 +239,7 @@ def test_one_loud_key_at_the_windows_edge(cuda_device, dtype, kernel, page_size,
     q, rows = _rounded(q, td), _rounded(rows, td)
     pool, table, mapping, _ = _pool(T, D, page_size, cuda_device, td)
     pool.view(-1, D)[mapping.long()] = rows.to(td).to(cuda_device)
-    q_len = 1 if kernel == "decode" else 40
+    q_len = 1 if "decode" in kernel else 40
     if window is not None:  # pages no query of the step sees are given back: whatever they hold must not matter
         lowest = max(0, T - q_len - window + 1)
         for block in range(lowest // page_size):
