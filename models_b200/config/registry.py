@@ -17,6 +17,7 @@ from .llama import ConfigError, LlamaConfig
 from .lovurax import ARCHITECTURE as LOVURAX, LovuraxConfig
 from .mabivik import ARCHITECTURE as MABIVIK, MabivikConfig
 from .rolevik import ARCHITECTURE as ROLEVIK, RolevikConfig
+from .rulunex import ARCHITECTURE as RULUNEX, RulunexConfig
 
 # name -> callable(raw config.json dict) -> object with .model_spec()
 _ARCHITECTURES: Dict[str, Callable[[Mapping[str, Any]], Any]] = {}
@@ -72,3 +73,4 @@ register_architecture(LOVURAX, LovuraxConfig.from_dict)
 register_architecture(KIVEZEN, KivezenConfig.from_dict)
 register_architecture(ROLEVIK, RolevikConfig.from_dict)
 register_architecture(MABIVIK, MabivikConfig.from_dict)
+register_architecture(RULUNEX, RulunexConfig.from_dict)

@@ -51,10 +51,14 @@ class RopeSpec:
 
 @dataclass(frozen=True)
 class NormSpec:
+    """x / sqrt(mean(x^2) + eps) * (gain_offset + weight): offset 0 for a weight stored as it is, 1 for one stored as its
+    distance from one."""
+
     size: int
     eps: float
     weights: Mapping[str, str] = field(default_factory=dict, hash=False, compare=False)
     kind: str = "rmsnorm"
+    gain_offset: float = 0.0
 
 
 @dataclass(frozen=True)
@@ -188,10 +192,21 @@ class ScheduleEntry:
     """One run of a layer.  The order in which layers run is a list of these: a layer may be
     named twice (its weights are shared, each run has a cache of its own) and a run may read the
     cache that an earlier run wrote (`cache_from` is that run's index in the schedule) instead of
-    writing one."""
+    writing one.  `joins`: before the run the residual stream passes the model's `join`."""
 
     layer: int
     cache_from: Optional[int] = None
+    joins: bool = False
+
+
+@dataclass(frozen=True)
+class StreamJoinSpec:
+    """The residual stream made anew from itself and the embedding's rows of the same tokens: x <- W [x; x_0] with one matrix
+    [width, 2 * width] (`weights`: weight).  The schedule's entries say where it happens."""
+
+    hidden_size: int
+    weights: Mapping[str, str] = field(default_factory=dict, hash=False, compare=False)
+    kind: str = "linear_join"
 
 
 @dataclass(frozen=True)
@@ -235,6 +250,7 @@ class ModelSpec:
     # Copies of the residual stream that the blocks keep side by side ([tokens, streams * width]); they all start as
     # the embedding's rows and are added up before the final norm.  1: the usual single stream.
     residual_streams: int = 1
+    join: Optional[StreamJoinSpec] = None  # what the schedule's entries with `joins` pass the stream through
     # Tensors a checkpoint of this architecture may hold that the model does not read: name patterns
     # (fnmatch) of buffers that are recomputed, and names that must repeat another tensor exactly (a
     # tied model's stored output matrix).  Anything else that is not asked for is an error.
@@ -247,6 +263,8 @@ class ModelSpec:
         for index, entry in enumerate(self.schedule):
             if not 0 <= entry.layer < len(self.layers):
                 raise ValueError(f"schedule[{index}] names layer {entry.layer}, the model has {len(self.layers)}")
+            if entry.joins and (self.join is None or self.residual_streams != 1):
+                raise ValueError(f"schedule[{index}] joins the stream with the embedding's rows: the model needs a join and one stream")
             if entry.cache_from is not None:
                 if not 0 <= entry.cache_from < index:
                     raise ValueError(
@@ -395,6 +413,16 @@ class ClampedExpertSpec:
 
 
 @dataclass(frozen=True)
+class ClampedFeedForwardSpec:
+    """One dense gated feed-forward with clamped branches (`weights`: gate, up, down)."""
+
+    hidden_size: int
+    expert: ClampedExpertSpec
+    weights: Mapping[str, str] = field(default_factory=dict, hash=False, compare=False)
+    kind: str = "clamped"
+
+
+@dataclass(frozen=True)
 class RoutedFeedForwardSpec:
     """A mixture of `num_experts` feed-forwards of one shape (`expert`): router logits z = router . x in float32; every
     token uses the `top` experts with the largest logits (ties to the lower index) with the softmax over the chosen
@@ -449,8 +477,9 @@ class ChunkedAttentionSpec:
     """Causal grouped-query softmax attention whose projections are normalised as a whole.  q, k and v have biases when
     `bias` is set; with `projection_norm` q (all heads side by side) passes ONE RMS norm with a gain of that size and eps `eps`,
     and so does k, before the heads are split and rotated (`position`, or None).  score = scale * q.k.  `chunk` n: query i sees
-    key j <= i only if floor(i / n) = floor(j / n), chunks counted from position 0 of the sequence (None: every earlier key).
-    Keys have `head_dim` coordinates, values `value_dim`."""
+    key j <= i only if floor(i / n) = floor(j / n), chunks counted from position 0 of the sequence (None: every earlier key);
+    `window` n: only if i - j < n.  Keys have `head_dim` coordinates, values `value_dim`.  `values_from_keys`: there is no value
+    matrix; a head's values are its keys as projected, before norm and rotation."""
 
     hidden_size: int
     num_heads: int
@@ -465,6 +494,8 @@ class ChunkedAttentionSpec:
     projection_norm: bool
     weights: Mapping[str, str] = field(default_factory=dict, hash=False, compare=False)
     kind: str = "chunked_attention"
+    window: Optional[int] = None
+    values_from_keys: bool = False
 
 
 @dataclass(frozen=True)

@@ -506,6 +506,27 @@ __global__ void store_rows_kernel(const float* __restrict__ src, Out* __restrict
         Num<Out>::store(dst + i, src[i]);
 }
 
+// The rows src [rows][width] stored in another type as column slices of wider tensors: dst, and copy where it is given (both with
+// row stride `stride`).  kVec elements a thread (4: width and strides multiples of 4, aligned slices).
+template <typename Out, int kVec>
+__global__ void store_columns_kernel(const float* __restrict__ src, Out* __restrict__ dst, Out* __restrict__ copy, int width, int stride, size_t total) {
+    grid_launch_dependents();
+    grid_dependency_wait();
+    const int per_row = width / kVec;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+        const size_t row = i / per_row, at = row * stride + (i % per_row) * kVec;
+        if (kVec == 4) {
+            const float4 v = load4(src + i * 4);
+            store4(dst + at, v);
+            if (copy != nullptr) store4(copy + at, v);
+        } else {
+            const float v = src[i];
+            Num<Out>::store(dst + at, v);
+            if (copy != nullptr) Num<Out>::store(copy + at, v);
+        }
+    }
+}
+
 // Eight elements a thread (columns and strides are multiples of 8 and the slices start on 16 bytes; 32 for float).
 template <typename T>
 __global__ void activate_vec8_kernel(const T* __restrict__ src, int src_stride, T* __restrict__ dst, int dst_stride, int cols8,
@@ -783,6 +804,27 @@ MB_EXPORT int mb_store_rows(const float* src, void* dst, int dtype, size_t total
     else
         return fail("store_rows: unknown dtype code %d", dtype);
     return check_launch("store_rows");
+}
+
+template <typename Out>
+static int launch_store_columns(const float* src, void* dst, void* copy, int rows, int width, int stride, cudaStream_t stream) {
+    const size_t align = 4 * sizeof(Out) - 1;
+    const bool vec = width % 4 == 0 && stride % 4 == 0 && !((uintptr_t)src & 15) && !((uintptr_t)dst & align) && !((uintptr_t)copy & align);
+    const size_t total = (size_t)rows * width / (vec ? 4 : 1), blocks = (total + 255) / 256;
+    const int grid = (int)(blocks > 148 * 32 ? 148 * 32 : blocks);
+    if (vec)
+        MB_LAUNCH("store_columns", (store_columns_kernel<Out, 4>), dim3(grid), dim3(256), 0, stream, true, src, (Out*)dst, (Out*)copy, width, stride, total);
+    else
+        MB_LAUNCH("store_columns", (store_columns_kernel<Out, 1>), dim3(grid), dim3(256), 0, stream, true, src, (Out*)dst, (Out*)copy, width, stride, total);
+    return check_launch("store_columns");
+}
+
+// src: float [rows][width], contiguous; dst, copy (or null): column slices with one row stride (in elements).
+MB_EXPORT int mb_store_columns(const float* src, void* dst, void* copy, int dtype, int rows, int width, int stride, cudaStream_t stream) {
+    if (rows <= 0 || width <= 0) return 0;
+    if (dtype == MB_F32) return launch_store_columns<float>(src, dst, copy, rows, width, stride, stream);
+    if (dtype == MB_BF16) return launch_store_columns<__nv_bfloat16>(src, dst, copy, rows, width, stride, stream);
+    return fail("store_columns: unknown dtype code %d", dtype);
 }
 
 // dst[r, c] = scale * act(src[r, c]) for [rows, cols] column slices with row strides (in elements); activation: MB_ACT_*.

@@ -35,6 +35,7 @@ class DecoderModel:
         self.final_norm = build_part("norm", spec.final_norm, runtime)
         self.embedding = build_part("embedding", spec.embedding, runtime)
         self.head = build_part("head", spec.head, runtime)
+        self.join = build_part("join", spec.join, runtime) if spec.join is not None else None
         # when set, called with (run index, a copy of the float32 residual stream after that run), for
         # finding the layer where two computations part (the reference's LayerObserver,
         # backend-java/.../llama/LlamaForwardPass.java:44-47,1179-1181)
@@ -49,6 +50,8 @@ class DecoderModel:
             requests += block.parameters()
         requests += self.final_norm.parameters()
         requests += self.head.parameters()
+        if self.join is not None:
+            requests += self.join.parameters()
         return _collect(requests)
 
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
@@ -60,6 +63,8 @@ class DecoderModel:
         self.final_norm.load(tensors)
         # tied output: the embedding matrix stands in (backend-java/.../llama/LlamaWeights.java:83-89)
         self.head.load(tensors, tied_to=getattr(self.embedding, "weight", None) if self.spec.head.tied else None)
+        if self.join is not None:
+            self.join.load(tensors)
         if self.runtime.mode == "bfloat16" and self.runtime.device.type == "cuda":
             from .fused_decode import FusedDecode
 
@@ -88,16 +93,25 @@ class DecoderModel:
             x = ops.stream_copies(x, streams)  # [tokens, streams * width]: every copy starts as the embedding's row
         pending = None
         schedule = self.spec.schedule
+        if self.join is not None:
+            self.join.begin(x, at_once=schedule[0].joins)
         for index, (run, entry) in enumerate(zip(runs, schedule)):
             block = self.blocks[entry.layer]
+            if entry.joins:
+                if as_delta(pending) is not None:
+                    ops.residual_add(x, as_delta(pending))
+                x, pending = self.join.forward(x, pending), None
+            after = schedule[index + 1] if index + 1 < len(schedule) else None
             if getattr(block, "takes_next_norm", False):
-                # the norm that reads the stream after this run: the next run's first norm, or the final one
-                following = self.blocks[schedule[index + 1].layer] if index + 1 < len(schedule) else None
-                next_norm = getattr(following, "mixer_norm", None) if following is not None else self.final_norm
+                # what reads the stream after this run: a join, the next run's first norm, or the final norm
+                if after is None:
+                    next_norm = self.final_norm
+                else:
+                    next_norm = self.join if after.joins else getattr(self.blocks[after.layer], "mixer_norm", None)
                 pending = block.forward(x, pending, batch, run, next_norm)
             elif getattr(block, "takes_next_block", False):
                 # the block that reads the streams after this run (none after the last one): its reading may ride in this one's writing
-                following = self.blocks[schedule[index + 1].layer] if index + 1 < len(schedule) else None
+                following = self.blocks[after.layer] if after is not None and not after.joins else None
                 pending = block.forward(x, pending, batch, run, following)
             else:
                 pending = block.forward(x, as_delta(pending), batch, run)
@@ -105,6 +119,8 @@ class DecoderModel:
                 delta = as_delta(pending)
                 seen = ops.stream_sum(x, self.spec.hidden_size) if streams > 1 else x
                 self.observer(run.run, seen + delta.float() if delta is not None else seen.clone())
+        if self.join is not None:
+            self.join.end()
         if batch.num_wanted == 0:
             return None
         if streams > 1:

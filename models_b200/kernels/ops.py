@@ -341,6 +341,20 @@ def store_rows(x: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
     return out
 
 
+def store_columns(x: torch.Tensor, dst: torch.Tensor, copy: Optional[torch.Tensor] = None) -> None:
+    """The float32 rows x stored in dst's type as a column slice of a wider tensor; `copy`: a second slice of the same tensor."""
+    _cuda(x, dst, copy)
+    if x.dtype != torch.float32 or x.dim() != 2 or not x.is_contiguous():
+        raise KernelError("store_columns: the rows must be contiguous float32")
+    for t in (dst, copy):
+        if t is not None:
+            _columns(t, "store_columns")
+            if t.shape != x.shape or t.dtype != dst.dtype or t.stride(0) != dst.stride(0):
+                raise KernelError(f"store_columns: {tuple(t.shape)} {t.dtype} does not take rows of {tuple(x.shape)}")
+    lib = elementwise()
+    _run(lib, lib.mb_store_columns(_p(x), _p(dst), _p(copy), _code(dst.dtype), x.shape[0], x.shape[1], dst.stride(0), _stream()))
+
+
 def result_norm_library():
     return load_library("mb_result_norm", ["result_norm.cu"])
 

@@ -1,11 +1,14 @@
-"""Grouped-query softmax attention whose projections are normalised as a whole and whose visibility is cut into chunks.
+"""Grouped-query softmax attention whose projections are normalised as a whole and whose visibility is cut into chunks or by
+a sliding window.
 
 q = Wq.xn + bq, k = Wk.xn + bk, v = Wv.xn + bv; with `projection_norm` the whole row q (all heads side by side) passes ONE RMS
 norm with a gain of that size, and so does k, before the heads are split; every head's first coordinates are then rotated by the
 token's position (the spec's `position`); score(i, j) = scale * q_i.k_j; with `chunk` n, query i sees key j <= i only if
-floor(i / n) = floor(j / n), chunks counted from position 0 of the sequence whatever the step's cut; softmax over the visible
+floor(i / n) = floor(j / n), chunks counted from position 0 of the sequence whatever the step's cut; with `window` n, only
+if i - j < n; softmax over the visible
 keys; head h reads the keys and values of head h / (heads / kv_heads); then Wo.  Biases, norms, rotation, scores and weights
-are float32 arithmetic in both modes.
+are float32 arithmetic in both modes.  With `values_from_keys` there is no Wv: the values are the projected keys before norm and
+rotation, so the cache keeps both forms of one projection.
 """
 
 from __future__ import annotations
@@ -28,6 +31,10 @@ class ChunkedAttentionMixer(SplitPart, Mixer):
             raise ValueError(f"{spec.num_heads} heads are no multiple of {spec.num_kv_heads} kv heads")
         if spec.chunk is not None and spec.chunk < 1:
             raise ValueError(f"a chunk holds at least one position, got {spec.chunk}")
+        if spec.window is not None and (spec.window < 1 or spec.chunk is not None):
+            raise ValueError(f"a window holds at least one position and goes without chunks, got {spec.window} and {spec.chunk}")
+        if spec.values_from_keys and (spec.value_dim != spec.head_dim or spec.bias):
+            raise ValueError("values that are the projected keys have the keys' size and no bias")
         self.q_width = spec.num_heads * spec.head_dim
         self.k_width = spec.num_kv_heads * spec.head_dim
         self.v_width = spec.num_kv_heads * spec.value_dim
@@ -41,10 +48,14 @@ class ChunkedAttentionMixer(SplitPart, Mixer):
                 runtime.shared[key] = build_part("position", spec.position, runtime)
             self.position = runtime.shared[key]
 
+    def _first(self):
+        return ("q", "k") if self.spec.values_from_keys else ("q", "k", "v")
+
     def parameters(self):
         s, n = self.spec, self.spec.weights
-        out = [ParamRequest(n["q"], (self.q_width, s.hidden_size)), ParamRequest(n["k"], (self.k_width, s.hidden_size)),
-               ParamRequest(n["v"], (self.v_width, s.hidden_size)), ParamRequest(n["o"], (s.hidden_size, self.mid_width))]
+        widths = {"q": self.q_width, "k": self.k_width, "v": self.v_width}
+        out = [ParamRequest(n[r], (widths[r], s.hidden_size)) for r in self._first()]
+        out.append(ParamRequest(n["o"], (s.hidden_size, self.mid_width)))
         if s.bias:
             out += [ParamRequest(n["q_bias"], (self.q_width,), "bias"), ParamRequest(n["k_bias"], (self.k_width,), "bias"),
                     ParamRequest(n["v_bias"], (self.v_width,), "bias")]
@@ -54,7 +65,7 @@ class ChunkedAttentionMixer(SplitPart, Mixer):
 
     def load(self, tensors):
         s, n, rt = self.spec, self.spec.weights, self.runtime
-        first = [rt.matrix(tensors[n[r]]) for r in ("q", "k", "v")]
+        first = [rt.matrix(tensors[n[r]]) for r in self._first()]
         if len({m.dtype for m in first}) > 1:
             first = [m.float() for m in first]
         self.w_in, self.starts = stack_rows(first)
@@ -70,7 +81,7 @@ class ChunkedAttentionMixer(SplitPart, Mixer):
 
     def kv_request(self):
         s = self.spec
-        return KvRequest(s.num_kv_heads, s.head_dim, None, s.value_dim)
+        return KvRequest(s.num_kv_heads, s.head_dim, s.window, s.value_dim)
 
     def inner(self, proj: torch.Tensor, mid: torch.Tensor, batch, run: RunContext, scale: float = 1.0) -> None:
         s, pos = self.spec, self.position
@@ -84,12 +95,13 @@ class ChunkedAttentionMixer(SplitPart, Mixer):
         at = self.starts
         q = proj[:, at[0]:at[0] + self.q_width]
         k = proj[:, at[1]:at[1] + self.k_width]
-        v = proj[:, at[2]:at[2] + self.v_width]
+        v = k if s.values_from_keys else proj[:, at[2]:at[2] + self.v_width]  # (k's columns themselves are not rewritten)
         ops.project_norm_rotate_store(q, k, v, *self.biases, *self.gains, s.eps, batch.positions, pos.cos if pos else None,
                                       pos.sin if pos else None, pos.rotary_dim if pos else 0, pos.interleaved if pos else False,
                                       run.k_pool, run.v_pool, group.slot_mapping, s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim)
         ops.gated_attention(q, mid, run.k_pool, run.v_pool, group.block_table, batch.cu_q, batch.kv_lens, batch.max_q_len,
-                            s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim, "softmax", s.scale, block=s.chunk or 0)
+                            s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim, "softmax", s.scale, block=s.chunk or 0,
+                            window=s.window or 0)
 
 
 register_part("mixer", "chunked_attention", ChunkedAttentionMixer)

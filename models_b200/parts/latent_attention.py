@@ -11,7 +11,9 @@ norm, the scores and the softmax are float32 in both modes.
 Variations (the spec says which).  Queries from a latent of their own, q = Uq.rmsnorm(Wdq.xn).  A position: every query head has
 `rotary_dim` coordinates more and the cached row as many more, one rotated key part that all heads share; the query in the latent
 space is [Uk_h^T q | rotated part], the cached row [c | rotated part], and their product is the whole score; the values are the
-row's first latent_dim numbers.  A window.  A gate per element.  Rows that another run cached (`own_rows` False).
+row's first latent_dim numbers.  (Rotated pairs (2i, 2i + 1) are brought side by side when the weights are loaded: the rotated
+parts meet in dot products only, so the order of their coordinates is nobody's business but theirs, and the kernels know one
+pairing.)  A window.  A gate per element.  Rows that another run cached (`own_rows` False).
 """
 
 from __future__ import annotations
@@ -38,8 +40,6 @@ class LatentAttentionMixer(SplitPart, Mixer):
         self.mid_width = spec.num_heads * spec.value_dim
         self.rope = None
         if spec.position is not None:
-            if spec.position.pairing != "half":
-                raise ValueError("the rotated part of a latent attention pairs coordinate i with i + rotary_dim / 2")
             key = ("position", spec.position, runtime.max_positions)
             if key not in runtime.shared:
                 runtime.shared[key] = build_part("position", spec.position, runtime)
@@ -55,6 +55,16 @@ class LatentAttentionMixer(SplitPart, Mixer):
             out.append(("gate", s.num_heads if s.gate_kind == "head" else self.mid_width))
         return out
 
+    def _paired(self, matrix: torch.Tensor, parts: int) -> torch.Tensor:
+        """The rows of `parts` equal parts, each ending in the rotated coordinates, with those ordered as pairs
+        (i, i + rotary_dim / 2)."""
+        if not self.turned or self.spec.position.pairing == "half":
+            return matrix
+        size = matrix.shape[0] // parts
+        kept = size - self.turned
+        order = list(range(kept)) + list(range(kept, size, 2)) + list(range(kept + 1, size, 2))
+        return matrix.view(parts, size, -1)[:, torch.tensor(order, device=matrix.device)].reshape(matrix.shape).contiguous()
+
     def parameters(self):
         s, n = self.spec, self.spec.weights
         out = [ParamRequest(n[role], (rows, s.hidden_size)) for role, rows in self._first()]
@@ -69,7 +79,9 @@ class LatentAttentionMixer(SplitPart, Mixer):
 
     def load(self, tensors):
         s, n, rt = self.spec, self.spec.weights, self.runtime
+        parts = {"q": s.num_heads, "down": 1}  # which of the first matrices end in rotated rows, and how often
         first = [rt.matrix(tensors[n[role]]) for role, _ in self._first()]
+        first = [self._paired(m, parts[role]) if role in parts else m for m, (role, _) in zip(first, self._first())]
         if len({m.dtype for m in first}) > 1:
             first = [m.float() for m in first]
         self.w_in, starts = stack_rows(first)
@@ -78,7 +90,7 @@ class LatentAttentionMixer(SplitPart, Mixer):
         self.latent_gain = rt.vector(tensors[n["down_norm"]]) if s.own_rows else None
         if s.query_latent:
             self.query_gain = rt.vector(tensors[n["down_q_norm"]])
-            self.up_q, _, _ = stack_columns([rt.matrix(tensors[n["up_q"]])])  # (columns of padding meet zeros)
+            self.up_q, _, _ = stack_columns([self._paired(rt.matrix(tensors[n["up_q"]]), s.num_heads)])  # (columns of padding meet zeros)
         dtype = rt.compute_dtype
         # per head: [latent_dim, head_dim] takes a query into the latent space, [value_dim, latent_dim] a result out of it
         self.into_latent = rt.matrix(tensors[n["up_k"]]).to(dtype).view(s.num_heads, s.head_dim, s.latent_dim).transpose(1, 2).contiguous()

@@ -1,7 +1,9 @@
 """RMSNorm fused with the residual add that precedes it.
 
 sumSq = sum x_i^2; rms = sqrt(sumSq/size + eps); out_i = x_i * (1/rms) * w_i
-(integrallis/models, backend-java/.../ops/TensorOps.java:45-58), all in float32.
+(integrallis/models, backend-java/.../ops/TensorOps.java:45-58), all in float32.  A weight stored as its distance from a
+constant (the spec's `gain_offset`) gets the constant added once, in float32, when it is loaded: whoever folds the norm reads
+`weight`, the gain itself.
 """
 
 from __future__ import annotations
@@ -21,10 +23,12 @@ class RmsNorm(Part):
     foldable = True
 
     def parameters(self):
-        return [ParamRequest(self.spec.weights["weight"], (self.spec.size,), "gain")]
+        return [ParamRequest(self.spec.weights["weight"], (self.spec.size,), "gain_offset" if self.spec.gain_offset else "gain")]
 
     def load(self, tensors):
         self.weight = self.runtime.vector(tensors[self.spec.weights["weight"]])
+        if self.spec.gain_offset:
+            self.weight = self.weight + self.spec.gain_offset
 
     def forward(self, x: torch.Tensor, delta: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
                 write_x: bool = True) -> torch.Tensor:

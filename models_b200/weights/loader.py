@@ -32,7 +32,8 @@ class WeightsError(ValueError):
 @dataclass(frozen=True)
 class ParamRequest:
     """A tensor a part needs.  kind: "matrix" (used by matrix products, random init N(0, std)),
-    "gain" (a norm's weight, random init 1 + N(0, gain_std)), "bias" (random init N(0, std)), "table" (integers in
+    "gain" (a norm's weight, random init 1 + N(0, gain_std)), "gain_offset" (a norm's weight stored as its distance from a
+    constant, random init N(0, gain_std)), "bias" (random init N(0, std)), "table" (integers in
     [0, limit), those of a row all different, random init uniform)."""
 
     name: str

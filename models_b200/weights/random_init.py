@@ -22,7 +22,8 @@ from .safetensors_io import write_safetensors
 
 def random_tensors(requests: Mapping[str, ParamRequest], seed: int, std: float = 0.02, gain_std: float = 0.1,
                    dtype: torch.dtype = torch.bfloat16, device="cpu") -> Dict[str, torch.Tensor]:
-    """Matrices and biases N(0, std); norm gains 1 + N(0, gain_std); tables int32, uniform.  Others drawn in float32, then rounded
+    """Matrices and biases N(0, std); norm gains 1 + N(0, gain_std) (those stored as a distance from a constant:
+    N(0, gain_std)); tables int32, uniform.  Others drawn in float32, then rounded
     to `dtype`.  Values come from a counter-based generator keyed by (seed, tensor name)
     (weights/philox_normal.py): on a CUDA device a kernel draws them in place, on the host numpy does,
     and both give the same bits."""
@@ -30,7 +31,7 @@ def random_tensors(requests: Mapping[str, ParamRequest], seed: int, std: float =
     device = torch.device(device)
     for name, request in requests.items():
         key = tensor_key(seed, name)
-        mean, scale = (1.0, gain_std) if request.kind == "gain" else (0.0, std)
+        mean, scale = {"gain": (1.0, gain_std), "gain_offset": (0.0, gain_std)}.get(request.kind, (0.0, std))
         shape = tuple(request.shape)
         count = 1
         for n in shape:
