@@ -21,6 +21,9 @@
 #define MB_ACT_GELU_TANH 1
 #define MB_ACT_RELU2 2
 #define MB_ACT_COUNT 3
+// A pair of branches with bounds (ClampedPair below) instead of act(gate) * up; its constants come in a host array of three
+// floats (limit, slope, up_offset) beside the code.
+#define MB_ACT_CLAMPED_SWISH 100
 
 namespace mb {
 
@@ -35,6 +38,26 @@ __device__ __forceinline__ float gate_activation(int activation, float z) {
     if (activation == MB_ACT_GELU_TANH)
         return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * z * (1.0f + 0.044715f * z * z)));
     return z / (1.0f + expf(-z));
+}
+
+// min(gate, limit) * sigmoid(slope * that) * (clamp(up, -limit, limit) + up_offset)
+struct ClampedPair {
+    float limit, slope, up_offset;
+};
+
+// What a gated product stores for a gate value and its up value.
+__device__ __forceinline__ float gated_pair(int activation, float gate, float up, const ClampedPair& clamp) {
+    if (activation == MB_ACT_CLAMPED_SWISH) {
+        const float g = fminf(gate, clamp.limit), u = fminf(fmaxf(up, -clamp.limit), clamp.limit);
+        return g / (1.0f + expf(-clamp.slope * g)) * (u + clamp.up_offset);
+    }
+    return gate_activation(activation, gate) * up;
+}
+
+// Whether a launcher knows the code; `clamp` (three floats on the host, or null) is copied out for the clamped form.
+inline bool gate_known(int activation, const float* clamp, ClampedPair* out) {
+    if (clamp != nullptr) *out = ClampedPair{clamp[0], clamp[1], clamp[2]};
+    return activation == MB_ACT_CLAMPED_SWISH ? clamp != nullptr : activation >= 0 && activation < MB_ACT_COUNT;
 }
 
 // The cluster barrier a block passes before it leaves, so that its shared memory outlives the other blocks' reads

@@ -136,10 +136,8 @@ struct GemmArgs {
     // reads (it is left out; its rows of the output are not written).  The table is written by a kernel before.
     const int* tile_group;    // null: a plain product
     int group_rows;           // rows of W per group (EPI_SWIGLU: gate rows; the up rows of the same group lie up_row_offset further)
-    float limit, slope, up_offset;  // activation kClampedSwish: min(gate, limit) * sigmoid(slope * that) * (clamp(up, -limit, limit) + up_offset)
+    ClampedPair clamp;        // EPI_SWIGLU with activation MB_ACT_CLAMPED_SWISH
 };
-
-constexpr int kClampedSwish = 100;  // (beside the MB_ACT_* codes; only the grouped entry point sets it)
 
 // kPair 1: a block works on a tile alone.  kPair 2: the two blocks of a cluster share a tile of 256 rows by BN columns
 // (tcgen05 cta_group::2): each loads its 128 rows of A and its half of the BN rows of W, the leader issues the products
@@ -468,14 +466,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                                 tmem_load_32_issue(taddr + 128 + c + 32 * part, u);
                                 tmem_load_wait();
 #pragma unroll
-                                for (int i = 0; i < 32; ++i) {
-                                    if (args.activation == kClampedSwish) {
-                                        const float g = fminf(v[i], args.limit), up = fminf(fmaxf(u[i], -args.limit), args.limit);
-                                        v[i] = g / (1.0f + expf(-args.slope * g)) * (up + args.up_offset);
-                                    } else {
-                                        v[i] = gate_activation(args.activation, v[i]) * u[i];
-                                    }
-                                }
+                                for (int i = 0; i < 32; ++i) v[i] = gated_pair(args.activation, v[i], u[i], args.clamp);
                             } else {
                                 tmem_load_32_issue(taddr + c + 32 * part, v);
                                 tmem_load_wait();
@@ -795,7 +786,7 @@ using namespace mb;
 // a: bfloat16 [m, k] (row stride lda); w: bfloat16 [n_w, k] (row stride ldw).
 // epilogue 0: out bfloat16 [m, n_w]; 1: out float32 [m, n_w]; 2: out float32 [m, n_w] += ; 3: w holds gate
 // rows [0, n_w/2) and up rows [n_w/2, n_w): out bfloat16 [m, n_w/2] = act(gate) * up, the activation code (MB_ACT_*)
-// in bits 8 and up of `epilogue`.
+// in bits 8 and up of `epilogue`; `clamp` (host, three floats) are the constants of MB_ACT_CLAMPED_SWISH, else null.
 // tile_width: 0 lets the launcher choose between 128 and 256 output columns per tile; the gated epilogue takes 256.
 // pair: 2 runs tiles of 256 rows x 256 columns on pairs of blocks (tcgen05 cta_group::2); 1: one block per tile; 0: the launcher chooses.
 // Scratch that always suffices for the ordered sum of the parts of K (residual epilogue): K is split only while
@@ -811,13 +802,14 @@ MB_EXPORT void mb_gemm_tcgen05_scratch(int multiprocessors, size_t* partial_floa
 // add into the stream as they finish, in no fixed order.
 MB_EXPORT int mb_gemm_tcgen05(const void* a, int lda, const void* w, int ldw, void* out, int ld_out, int m, int n_w, int k,
                               int epilogue, int multiprocessors, int tile_width, int pair, float* partial, int* tickets,
-                              cudaStream_t stream) {
+                              const float* clamp, cudaStream_t stream) {
     if (tile_width != 0 && tile_width != 128 && tile_width != 256) return fail("gemm_tcgen05: tile width %d is not built (128, 256)", tile_width);
     if (pair < 0 || pair > 2) return fail("gemm_tcgen05: pair must be 0, 1 or 2, got %d", pair);
     if (pair == 2 && tile_width == 128) return fail("gemm_tcgen05: pairs of blocks take tiles of 256 columns");
     const int activation = epilogue >> 8;
     epilogue &= 0xff;
-    if (activation < 0 || activation >= MB_ACT_COUNT) return fail("gemm_tcgen05: unknown gate activation code %d", activation);
+    GemmArgs args{};
+    if (!gate_known(activation, clamp, &args.clamp)) return fail("gemm_tcgen05: unknown gate activation code %d", activation);
     if (m <= 0 || n_w <= 0) return 0;
     if (k <= 0 || k % 8 || lda % 8 || ldw % 8) return fail("gemm_tcgen05: k (%d) and the row strides (%d, %d) must be multiples of 8", k, lda, ldw);
     if (((uintptr_t)a & 15) || ((uintptr_t)w & 15)) return fail("gemm_tcgen05: operands must start on 16-byte boundaries");
@@ -828,7 +820,6 @@ MB_EXPORT int mb_gemm_tcgen05(const void* a, int lda, const void* w, int ldw, vo
     CUtensorMap map_a, map_w;
     if (int status = make_map(&map_a, a, m, k, lda)) return status;
     if (int status = make_map(&map_w, w, n_w, k, ldw)) return status;
-    GemmArgs args{};
     args.m = m; args.n = n; args.k = k; args.up_row_offset = n; args.activation = activation; args.k_splits = 1;
     args.partial = partial; args.tickets = tickets; args.out = out; args.ld_out = ld_out;
     switch (epilogue) {
@@ -861,8 +852,8 @@ MB_EXPORT int mb_gemm_tcgen05_grouped(const void* a, int lda, const void* w, int
     if (int status = make_map(&map_a, a, m, k, lda)) return status;
     if (int status = make_map(&map_w, w, w_rows, k, ldw)) return status;
     GemmArgs args{};
-    args.m = m; args.n = n; args.k = k; args.up_row_offset = up_row_offset; args.activation = kClampedSwish; args.k_splits = 1;
-    args.out = out; args.ld_out = ld_out; args.tile_group = tile_group; args.group_rows = n; args.limit = limit; args.slope = slope; args.up_offset = up_offset;
+    args.m = m; args.n = n; args.k = k; args.up_row_offset = up_row_offset; args.activation = MB_ACT_CLAMPED_SWISH; args.k_splits = 1;
+    args.out = out; args.ld_out = ld_out; args.tile_group = tile_group; args.group_rows = n; args.clamp = ClampedPair{limit, slope, up_offset};
     if (gated) return launch_tile<EPI_SWIGLU, 256, 1>(map_a, map_w, args, multiprocessors, stream);
     return launch_tile<EPI_F32, 256, 1>(map_a, map_w, args, multiprocessors, stream);
 }

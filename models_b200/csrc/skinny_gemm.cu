@@ -48,7 +48,7 @@ namespace mb {
 using bf16 = __nv_bfloat16;
 
 enum { PRO_NONE = 0, PRO_NORM = 1, PRO_PRE = 2 };
-enum { EPI_BF16 = 0, EPI_F32 = 1, EPI_RESIDUAL = 2, EPI_SWIGLU = 3, EPI_ROPE = 4, EPI_TANH = 5, EPI_SIDE = 6 };
+enum { EPI_BF16 = 0, EPI_F32 = 1, EPI_RESIDUAL = 2, EPI_SWIGLU = 3, EPI_ROPE = 4, EPI_TANH = 5, EPI_SIDE = 6, EPI_PAIRS = 7 };
 
 constexpr int kWarps = 4;
 constexpr int kThreads = kWarps * 32;
@@ -125,6 +125,12 @@ struct SkinnyArgs {
     const bf16* side_table;    // [vocab][side_dim]
     const int* side_tokens;    // [batch]
     int side_dim;
+    // EPI_PAIRS: W holds plain_rows rows whose results are stored as they are (out_bf16), then pair_offset gate rows and as many up
+    // rows, whose pairs go to mid as gated_pair makes them
+    int plain_rows;
+    bf16* mid;                 // [batch][ld_mid]
+    int ld_mid;
+    ClampedPair clamp;         // EPI_PAIRS and EPI_SWIGLU, with activation MB_ACT_CLAMPED_SWISH
     const int* rows;      // optional: activation row b is xf row rows[b]
     bf16* out_bf16;
     float* out_f32;       // EPI_F32 output, or the residual stream for EPI_RESIDUAL
@@ -177,7 +183,9 @@ skinny_gemm_kernel(const SkinnyArgs args) {
     const int rank = args.k_split > 1 ? (int)cg::this_cluster().block_rank() : 0;
     const int cluster_id = blockIdx.x / args.k_split, clusters = gridDim.x / args.k_split;
     const int rows_total = EPI == EPI_SWIGLU ? args.pair_offset : (EPI == EPI_ROPE ? args.n / 2 : args.n);  // rows, or pairs
-    const int tiles_total = (rows_total + kTileRows - 1) / kTileRows;
+    // EPI_PAIRS: tiles of 16 plain rows, then tiles of 8 gate rows with their 8 up rows
+    const int plain_tiles = EPI == EPI_PAIRS ? (args.plain_rows + 15) / 16 : 0;
+    const int tiles_total = EPI == EPI_PAIRS ? plain_tiles + (args.pair_offset + 7) / 8 : (rows_total + kTileRows - 1) / kTileRows;
     const int tiles_mine = cluster_id < tiles_total ? (tiles_total - cluster_id + clusters - 1) / clusters : 0;
     // K: the block's part, then this warp's slice of it
     const int part_begin = rank * args.k_unit;
@@ -219,6 +227,9 @@ skinny_gemm_kernel(const SkinnyArgs args) {
             } else if (EPI == EPI_ROPE) {  // tile = (head, eighth of its first half); partner half a head further
                 const int tiles_per_head = args.head_dim / 16;
                 row = (tile / tiles_per_head) * args.head_dim + (tile % tiles_per_head) * 8 + group_id + h * (args.head_dim / 2);
+            } else if (EPI == EPI_PAIRS) {
+                row = tile < plain_tiles ? min(args.plain_rows - 1, tile * 16 + group_id + 8 * h)
+                                         : args.plain_rows + min(args.pair_offset - 1, (tile - plain_tiles) * 8 + group_id) + h * args.pair_offset;
             } else {
                 row = min(rows_total - 1, tile * 16 + group_id + 8 * h);
             }
@@ -444,7 +455,10 @@ skinny_gemm_kernel(const SkinnyArgs args) {
             const int row = tile * kTileRows + row_in_tile;
             const bool emits = EPI == EPI_RESIDUAL && args.emit_gain != nullptr;
             float squares = 0.0f;  // of the new x, where the next norm's rows are prepared
-            if (row >= rows_total || col >= args.batch) {
+            const bool pairs = EPI == EPI_PAIRS && tile >= plain_tiles;
+            const int pair = (tile - plain_tiles) * 8 + row_in_tile;
+            const bool outside = EPI == EPI_PAIRS ? (pairs ? row_in_tile >= 8 || pair >= args.pair_offset : row >= args.plain_rows) : row >= rows_total;
+            if (outside || col >= args.batch) {
                 if (!emits) continue;  // (with them, whole warps stay for the sums below)
             } else {
             float value = 0.0f, second = 0.0f;  // second: the up row that matches a gate row
@@ -452,7 +466,7 @@ skinny_gemm_kernel(const SkinnyArgs args) {
                 const float* from = args.k_split > 1 ? cg::this_cluster().map_shared_rank(mine, r) : mine;
                 for (int w = 0; w < kWarps; ++w) {
                     value += from[(w * 16 + row_in_tile) * COLS + col];
-                    if (kPaired) second += from[(w * 16 + row_in_tile + 8) * COLS + col];
+                    if (kPaired || pairs) second += from[(w * 16 + row_in_tile + 8) * COLS + col];
                 }
             }
             if (PRO == PRO_NORM) {
@@ -500,7 +514,11 @@ skinny_gemm_kernel(const SkinnyArgs args) {
                 if (i != (int)threadIdx.x) e = row < args.side_dim ? __bfloat162float(args.side_table[(size_t)args.side_tokens[col] * args.side_dim + row]) : 0.0f;
                 args.out_bf16[at] = __float2bfloat16_rn(row < args.side_dim ? gate_activation(MB_ACT_GELU_TANH, value) * e : 0.0f);
             }
-            if (EPI == EPI_SWIGLU) args.out_bf16[at] = __float2bfloat16_rn(gate_activation(args.activation, value) * second);
+            if (EPI == EPI_SWIGLU) args.out_bf16[at] = __float2bfloat16_rn(gated_pair(args.activation, value, second, args.clamp));
+            if (EPI == EPI_PAIRS) {
+                if (pairs) args.mid[(size_t)col * args.ld_mid + pair] = __float2bfloat16_rn(gated_pair(args.activation, value, second, args.clamp));
+                else args.out_bf16[at] = __float2bfloat16_rn(value);
+            }
             if (EPI == EPI_ROPE) {
                 const int tiles_per_head = args.head_dim / 16, half = args.head_dim / 2;
                 const int head = tile / tiles_per_head, d0 = (tile % tiles_per_head) * 8 + row_in_tile;
@@ -599,11 +617,11 @@ MB_EXPORT int mb_skinny_max_rows(int with_norm) { return with_norm ? 16 : 32; }
 // (MB_ACT_*) in bits 8 and up of `epilogue`.
 static int skinny_gemm(const void* w, int ldw, int n, int k, int batch, const void* x, int ldx, const float* xf,
                        int ldxf, const float* gain, float eps, const int* rows, void* out, int ld_out,
-                       int epilogue, int multiprocessors, int dependent, SkinnyArgs args, cudaStream_t stream) {
+                       int epilogue, int multiprocessors, int dependent, SkinnyArgs args, cudaStream_t stream, const float* clamp = nullptr) {
     if (batch <= 0 || n <= 0) return 0;
     const int activation = epilogue >> 8;
     epilogue &= 0xff;
-    if (activation < 0 || activation >= MB_ACT_COUNT) return fail("skinny_gemm: unknown gate activation code %d", activation);
+    if (!gate_known(activation, clamp, &args.clamp)) return fail("skinny_gemm: unknown gate activation code %d", activation);
     args.activation = activation;
     if (batch > 32) return fail("skinny_gemm: takes at most 32 activation rows, got %d", batch);
     if (k <= 0 || k % 8 || ldw % 8) return fail("skinny_gemm: k (%d) and the weight row stride (%d) must be multiples of 8", k, ldw);
@@ -616,7 +634,7 @@ static int skinny_gemm(const void* w, int ldw, int n, int k, int batch, const vo
     args.w = (const bf16*)w; args.ldw = ldw; args.n = n; args.k = k; args.batch = batch;
     args.x = (const bf16*)x; args.ldx = ldx; args.xf = xf; args.ldxf = ldxf; args.gain = gain; args.eps = eps; args.rows = rows;
     args.out_bf16 = (bf16*)out; args.out_f32 = (float*)out; args.ld_out = ld_out;
-    args.pair_offset = epilogue == EPI_SWIGLU ? n / 2 : 0;
+    if (epilogue != EPI_PAIRS) args.pair_offset = epilogue == EPI_SWIGLU ? n / 2 : 0;
     args.dependent = dependent;
     if (epilogue == EPI_SWIGLU) args.n = n / 2;
     // Planning.  A block's shared memory holds its activations (rows x k_unit bfloat16), the warps' rings
@@ -625,7 +643,8 @@ static int skinny_gemm(const void* w, int ldw, int n, int k, int batch, const vo
     // to fill idle multiprocessors was measured and lost to the cluster barrier it adds.  Blocks walk
     // several row tiles when there are more tiles than resident blocks.
     const int rows_total = (epilogue == EPI_SWIGLU || epilogue == EPI_ROPE) ? n / 2 : n;
-    const int tiles = (epilogue == EPI_SWIGLU || epilogue == EPI_ROPE) ? (rows_total + 7) / 8 : (rows_total + 15) / 16;
+    const int tiles = epilogue == EPI_PAIRS ? (args.plain_rows + 15) / 16 + (args.pair_offset + 7) / 8
+                      : (epilogue == EPI_SWIGLU || epilogue == EPI_ROPE) ? (rows_total + 7) / 8 : (rows_total + 15) / 16;
     const int cols = batch <= 8 ? 8 : (batch <= 16 ? 16 : 32);
     auto smem_for = [&](int split) {
         const int k_unit = ((k + split - 1) / split + kWarps * kStep - 1) / (kWarps * kStep) * (kWarps * kStep);
@@ -668,6 +687,9 @@ static int skinny_gemm(const void* w, int ldw, int n, int k, int batch, const vo
     MB_CASE(PRO_PRE, EPI_ROPE)
     MB_CASE(PRO_NONE, EPI_TANH)
     MB_CASE(PRO_NONE, EPI_SIDE)
+    MB_CASE(PRO_NONE, EPI_PAIRS)
+    MB_CASE(PRO_NORM, EPI_PAIRS)
+    MB_CASE(PRO_PRE, EPI_PAIRS)
 #undef MB_CASE
     return fail("skinny_gemm: no kernel for prologue %d with epilogue %d", prologue, epilogue);
 }
@@ -681,14 +703,29 @@ MB_EXPORT int mb_skinny_gemm(const void* w, int ldw, int n, int k, int batch, co
                              int ldxf, const float* gain, float eps, const int* rows, void* out, int ld_out,
                              int epilogue, int multiprocessors, int dependent, const float* ssq_parts, int ssq_count,
                              const float* emit_gain, void* emit_rows, int ld_emit, float* emit_ssq, int* parts_written,
-                             cudaStream_t stream) {
+                             const float* clamp, cudaStream_t stream) {
     if ((epilogue & 0xff) >= EPI_ROPE) return fail("skinny_gemm: epilogue %d has an entry point of its own", epilogue & 0xff);
     SkinnyArgs args{};
     args.ssq_parts = ssq_parts; args.ssq_count = ssq_count;
     args.emit_gain = emit_gain; args.emit_rows = (bf16*)emit_rows; args.ld_emit = ld_emit; args.emit_ssq = emit_ssq;
     if (parts_written) *parts_written = (n + 15) / 16;
     return skinny_gemm(w, ldw, n, k, batch, x, ldx, xf, ldxf, gain, eps, rows, out, ld_out, epilogue, multiprocessors, dependent,
-                       args, stream);
+                       args, stream, clamp);
+}
+
+// One product for a matrix of two kinds of rows: `plain_rows` rows whose results are stored as they are (out, bfloat16, row stride
+// ld_out), then `pairs` gate rows and as many up rows, whose gated pairs go to mid (bfloat16 [batch, pairs], row stride ld_mid).
+// activation: MB_ACT_* or MB_ACT_CLAMPED_SWISH with its constants in `clamp` (host, three floats).
+MB_EXPORT int mb_skinny_gemm_pairs(const void* w, int ldw, int plain_rows, int pairs, int k, int batch, const void* x, int ldx, const float* xf,
+                                   int ldxf, const float* gain, float eps, void* out, int ld_out, void* mid, int ld_mid, int activation,
+                                   const float* clamp, int multiprocessors, int dependent, const float* ssq_parts, int ssq_count,
+                                   cudaStream_t stream) {
+    if (plain_rows <= 0 || pairs <= 0 || !out || !mid) return fail("skinny_gemm_pairs: %d plain rows and %d pairs need both outputs", plain_rows, pairs);
+    SkinnyArgs args{};
+    args.plain_rows = plain_rows; args.pair_offset = pairs; args.mid = (bf16*)mid; args.ld_mid = ld_mid;
+    args.ssq_parts = ssq_parts; args.ssq_count = ssq_count;
+    return skinny_gemm(w, ldw, plain_rows + 2 * pairs, k, batch, x, ldx, xf, ldxf, gain, eps, nullptr, out, ld_out, EPI_PAIRS | (activation << 8),
+                       multiprocessors, dependent, args, stream, clamp);
 }
 
 // x_out += sigmoid(gate + gate_bias) * (x . w^T): the residual epilogue with a gate on what is added.  gate: bfloat16

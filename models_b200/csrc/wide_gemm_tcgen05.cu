@@ -40,6 +40,7 @@ struct WideArgs {
     int rows_total;       // output columns = weight rows (EPI_SWIGLU: gate rows)
     int up_row_offset;    // EPI_SWIGLU: first up row of W
     int activation;       // EPI_SWIGLU: the gate's activation (MB_ACT_*)
+    ClampedPair clamp;    // EPI_SWIGLU with MB_ACT_CLAMPED_SWISH
     int batch, k;
     int splits;           // blocks of a cluster that share a tile, each with its own part of K
     int k_blocks_per_split;
@@ -357,8 +358,8 @@ wide_gemm_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
                 up.x *= scale; up.y *= scale; up.z *= scale; up.w *= scale;
                 const int a = args.activation;
                 *reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(args.out) + (size_t)col * args.ld_out + row) =
-                    make_uint2(pack_bf16(gate_activation(a, gate.x) * up.x, gate_activation(a, gate.y) * up.y),
-                               pack_bf16(gate_activation(a, gate.z) * up.z, gate_activation(a, gate.w) * up.w));
+                    make_uint2(pack_bf16(gated_pair(a, gate.x, up.x, args.clamp), gated_pair(a, gate.y, up.y, args.clamp)),
+                               pack_bf16(gated_pair(a, gate.z, up.z, args.clamp), gated_pair(a, gate.w, up.w, args.clamp)));
             } else {  // EPI_ROPE: pairs `unit`.. of the tile are coordinates d and d + head/2 of one of its heads
                 const int hd = args.head_dim, half = hd / 2;
                 const int head_in_tile = unit / half, d0 = unit % half;
@@ -495,18 +496,19 @@ using namespace mb;
 // ssq_parts (or null): [ssq_count][128] parts of the sums of squares of the rows that x is the gained copy of; the
 // results are then scaled by 1 / sqrt(sum / norm_width + eps).  emit_gain (or null, epilogue 2 only): the next norm's
 // gain; the new x times it goes to emit_rows (bfloat16, row stride ld_emit), the blocks' parts of the new rows' sums of
-// squares to emit_ssq [parts][128], and *parts_written says how many parts there are.
+// squares to emit_ssq [parts][128], and *parts_written says how many parts there are.  clamp (host, three floats): the
+// constants of MB_ACT_CLAMPED_SWISH, else null.
 MB_EXPORT int mb_wide_gemm(const void* x, int ldx, const void* w, int ldw, void* out, int ld_out, int batch, int n_w, int k,
                            int epilogue, int multiprocessors, const float* ssq_parts, int ssq_count, int norm_width, float eps,
                            const float* emit_gain, void* emit_rows, int ld_emit, float* emit_ssq, int* parts_written,
-                           cudaStream_t stream) {
+                           const float* clamp, cudaStream_t stream) {
     if (batch <= 0 || n_w <= 0) return 0;
     const int activation = epilogue >> 8;
     epilogue &= 0xff;
-    if (activation < 0 || activation >= MB_ACT_COUNT) return fail("wide_gemm: unknown gate activation code %d", activation);
+    WideArgs args{};
+    if (!gate_known(activation, clamp, &args.clamp)) return fail("wide_gemm: unknown gate activation code %d", activation);
     if (int status = check_operands("wide_gemm", x, ldx, w, ldw, batch, k)) return status;
     if (epilogue == EPI_SWIGLU && n_w % 2) return fail("wide_gemm: the gated epilogue needs an even number of weight rows, got %d", n_w);
-    WideArgs args{};
     args.rows_total = epilogue == EPI_SWIGLU ? n_w / 2 : n_w;
     args.up_row_offset = args.rows_total;
     args.activation = activation;

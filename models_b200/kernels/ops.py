@@ -227,6 +227,16 @@ def gated_epilogue(activation: str = "silu") -> int:
     return EPI_SWIGLU | (activation_code(activation) << 8)
 
 
+EPI_CLAMPED = 3 | (100 << 8)  # EPI_SWIGLU with the clamped pair of csrc/common.cuh, whose constants come beside it (`clamp`)
+
+
+def _clamp_args(epilogue: int, clamp):
+    """The constants (limit, slope, up_offset) of a clamped epilogue as the C launchers take them, or None."""
+    if (epilogue == EPI_CLAMPED) != (clamp is not None):
+        raise KernelError("a clamped epilogue comes with its constants (limit, slope, up_offset), other epilogues without")
+    return None if clamp is None else (ctypes.c_float * 3)(*clamp)
+
+
 def swiglu(gate_up: torch.Tensor, activation: str = "silu") -> torch.Tensor:
     """act(gate) * up for a [rows, 2*width] tensor whose first half of columns is the gate."""
     _cuda(gate_up)
@@ -1569,13 +1579,15 @@ def multiprocessors(device) -> int:
 
 def skinny_gemm(weight: torch.Tensor, epilogue: int, x: Optional[torch.Tensor] = None, xf: Optional[torch.Tensor] = None,
                 gain: Optional[torch.Tensor] = None, eps: float = 0.0, rows: Optional[torch.Tensor] = None,
-                out: Optional[torch.Tensor] = None, norm_parts=None, emit_gain: Optional[torch.Tensor] = None):
+                out: Optional[torch.Tensor] = None, norm_parts=None, emit_gain: Optional[torch.Tensor] = None,
+                emit_rows: Optional[torch.Tensor] = None, clamp=None):
     """Few activation rows times weight^T ([n, k] bfloat16).  Activations: `x` (bfloat16 [rows, k]), or
     `xf` (the float32 residual rows, optionally gathered by `rows`) normalised on the fly with `gain`
     and `eps`.  Epilogues: EPI_BF16 / EPI_F32 store [rows, n]; EPI_RESIDUAL adds into `out` (float32
     [rows, n]); EPI_SWIGLU takes weight = [gate rows; up rows] and stores act(gate) * up [rows, n/2].
     `norm_parts` and `emit_gain` as for wide_gemm: `x` is then the rows times a norm's gain, divided by their
-    root mean square in the epilogue; a residual product can prepare the next norm's rows the same way."""
+    root mean square in the epilogue; a residual product can prepare the next norm's rows the same way.
+    EPI_CLAMPED: EPI_SWIGLU with a clamped pair, `clamp` = (limit, slope, up_offset)."""
     _cuda(weight, x, xf, gain, rows, out, emit_gain)
     n, k = weight.shape
     norm = gain is not None
@@ -1605,12 +1617,10 @@ def skinny_gemm(weight: torch.Tensor, epilogue: int, x: Optional[torch.Tensor] =
     ssq, count, _, _, part_eps = _norm_args(norm_parts, batch, SSQ_COLUMNS)
     if norm_parts is not None and norm_parts[2] != k:
         raise KernelError("the norm's width is the product's k")
-    emit_rows = emit_ssq = None
+    emit_ssq = None
     written = ctypes.c_int(0)
     if emit_gain is not None:
-        if kind != EPI_RESIDUAL or emit_gain.dtype != torch.float32 or emit_gain.numel() != n:
-            raise KernelError("the next norm's rows come from the residual epilogue, with a float32 gain of the output's width")
-        emit_rows = torch.empty((batch, n), dtype=torch.bfloat16, device=weight.device)
+        emit_rows = _emitted_rows(kind, emit_gain, emit_rows, batch, n, weight.device)
         emit_ssq = torch.empty((-(-n // 16), SSQ_COLUMNS), dtype=torch.float32, device=weight.device)
     lib = skinny()
     _run(lib, lib.mb_skinny_gemm(_p(weight), weight.stride(0), n, k, batch, _p(x), x.stride(0) if x is not None else 0,
@@ -1618,9 +1628,58 @@ def skinny_gemm(weight: torch.Tensor, epilogue: int, x: Optional[torch.Tensor] =
                                  part_eps if norm_parts is not None else ctypes.c_float(eps), _p(rows),
                                  _p(out), out.stride(0), epilogue, _sm_count(weight.device), 1, ssq, count, _p(emit_gain),
                                  _p(emit_rows), emit_rows.stride(0) if emit_rows is not None else 0, _p(emit_ssq),
-                                 ctypes.byref(written), _stream()))
+                                 ctypes.byref(written), _clamp_args(epilogue, clamp), _stream()))
     if emit_gain is not None:
         return out, emit_rows, emit_ssq, written.value
+    return out
+
+
+def _emitted_rows(kind: int, emit_gain: torch.Tensor, emit_rows: Optional[torch.Tensor], batch: int, n: int, device) -> torch.Tensor:
+    """Where a residual product leaves the rows of the next norm: a new tensor, or the column slice given."""
+    if kind != EPI_RESIDUAL or emit_gain.dtype != torch.float32 or emit_gain.numel() != n:
+        raise KernelError("the next norm's rows come from the residual epilogue, with a float32 gain of the output's width")
+    if emit_rows is None:
+        return torch.empty((batch, n), dtype=torch.bfloat16, device=device)
+    _columns(emit_rows, "emit_rows")
+    if emit_rows.dtype != torch.bfloat16 or tuple(emit_rows.shape) != (batch, n) or emit_rows.stride(0) % 4 or emit_rows.data_ptr() % 8:
+        raise KernelError(f"the next norm's rows need an aligned bfloat16 slice [{batch}, {n}], got {tuple(emit_rows.shape)} {emit_rows.dtype}")
+    return emit_rows
+
+
+def skinny_gemm_pairs(weight: torch.Tensor, plain_rows: int, mid: torch.Tensor, clamp, x: Optional[torch.Tensor] = None,
+                      xf: Optional[torch.Tensor] = None, gain: Optional[torch.Tensor] = None, eps: float = 0.0, norm_parts=None) -> torch.Tensor:
+    """The decode product over a matrix of two kinds of rows, [plain_rows; gate rows; up rows] (bfloat16 [n, k]): the plain rows'
+    results come back as bfloat16 [rows, plain_rows]; the gate/up pairs go to `mid` (bfloat16 [rows, pairs], a column slice is fine)
+    as min(gate, limit) * sigmoid(slope * that) * (clamp(up, -limit, limit) + up_offset), `clamp` = (limit, slope, up_offset).
+    Activations as for skinny_gemm: `x`, or `xf` normalised with `gain` and `eps`, or `x` with `norm_parts`."""
+    _cuda(weight, x, xf, gain, mid)
+    n, k = weight.shape
+    norm = gain is not None
+    if norm:
+        if xf is None or xf.dtype != torch.float32 or xf.stride(1) != 1 or xf.shape[1] != k or gain.dtype != torch.float32 or gain.numel() != k:
+            raise KernelError("the norm prologue needs float32 rows and a float32 gain of the weight's width")
+        if norm_parts is not None:
+            raise KernelError("a product normalises float32 rows itself or takes rows with parts of their sums of squares, not both")
+    elif x is None or x.dtype != torch.bfloat16 or x.stride(1) != 1 or x.shape[1] != k:
+        raise KernelError("activations must be bfloat16 rows of the weight's width")
+    batch = (xf if norm else x).shape[0]
+    _columns(mid, "mid")
+    pairs = mid.shape[1]
+    if plain_rows <= 0 or plain_rows + 2 * pairs != n or not skinny_takes(weight, batch, norm or norm_parts is not None):
+        raise KernelError(f"skinny_gemm_pairs: {plain_rows} rows and {pairs} pairs do not make a {tuple(weight.shape)} {weight.dtype} weight, or it is not taken")
+    if mid.dtype != torch.bfloat16 or mid.shape[0] != batch:
+        raise KernelError(f"skinny_gemm_pairs: the pairs' results are bfloat16 [{batch}, {pairs}], got {tuple(mid.shape)} {mid.dtype}")
+    ssq, count, width, part_eps = None, 0, k, ctypes.c_float(eps)
+    if norm_parts is not None:
+        ssq, count, _, width, part_eps = _norm_args(norm_parts, batch, SSQ_COLUMNS)
+    if width != k:
+        raise KernelError("the norm's width is the product's k")
+    out = torch.empty((batch, plain_rows), dtype=torch.bfloat16, device=weight.device)
+    lib = skinny()
+    _run(lib, lib.mb_skinny_gemm_pairs(_p(weight), weight.stride(0), int(plain_rows), pairs, k, batch, _p(x), x.stride(0) if x is not None else 0,
+                                       _p(xf), xf.stride(0) if xf is not None else 0, _p(gain), part_eps, _p(out), out.stride(0), _p(mid),
+                                       mid.stride(0), EPI_CLAMPED >> 8, _clamp_args(EPI_CLAMPED, clamp), _sm_count(weight.device), 1, ssq, count,
+                                       _stream()))
     return out
 
 
@@ -1743,7 +1802,7 @@ _split_tickets = {}
 
 
 def gemm_tcgen05(a: torch.Tensor, weight: torch.Tensor, epilogue: int = EPI_BF16, out: Optional[torch.Tensor] = None,
-                 tile_width: int = 0, pair: int = 0, arrival_order: bool = False) -> torch.Tensor:
+                 tile_width: int = 0, pair: int = 0, arrival_order: bool = False, clamp=None) -> torch.Tensor:
     """a [m, k] . weight[n, k]^T on the tcgen05 tensor cores (bfloat16 in, float accumulation).
     Epilogues as for skinny_gemm: EPI_BF16 / EPI_F32 store, EPI_RESIDUAL adds into `out` (float32
     [m, n]), EPI_SWIGLU stores act(gate) * up for weight = [gate rows; up rows].  tile_width 0 lets
@@ -1779,7 +1838,7 @@ def gemm_tcgen05(a: torch.Tensor, weight: torch.Tensor, epilogue: int = EPI_BF16
             # zero once; every launch leaves the tickets at zero
             tickets = _split_tickets[key] = torch.zeros((need_tickets.value,), dtype=torch.int32, device=a.device)
     _run(lib, lib.mb_gemm_tcgen05(_p(a), a.stride(0), _p(weight), weight.stride(0), _p(out), out.stride(0), m, n_w, k,
-                                  epilogue, sms, tile_width, pair, _p(partial), _p(tickets), _stream()))
+                                  epilogue, sms, tile_width, pair, _p(partial), _p(tickets), _clamp_args(epilogue, clamp), _stream()))
     return out
 
 
@@ -1841,7 +1900,7 @@ def _norm_args(norm_parts, rows: int, columns: Optional[int] = None):
 
 
 def wide_gemm(x: torch.Tensor, weight: torch.Tensor, epilogue: int = EPI_BF16, out: Optional[torch.Tensor] = None,
-              norm_parts=None, emit_gain: Optional[torch.Tensor] = None):
+              norm_parts=None, emit_gain: Optional[torch.Tensor] = None, emit_rows: Optional[torch.Tensor] = None, clamp=None):
     """Up to 128 activation rows times weight^T on the tcgen05 tensor cores with the weights as the
     128-row operand (decode at wide batches); K is split over the blocks of a cluster where a matrix has
     few row tiles, their sums meeting in distributed shared memory in a fixed order.  Epilogues as for
@@ -1866,18 +1925,17 @@ def wide_gemm(x: torch.Tensor, weight: torch.Tensor, epilogue: int = EPI_BF16, o
             raise KernelError("the residual epilogue adds into a float32 [rows, n] tensor")
     elif out is None:
         out = torch.empty((batch, n), dtype=torch.float32 if kind == EPI_F32 else torch.bfloat16, device=x.device)
-    emit_rows = emit_ssq = None
+    emit_ssq = None
     written = ctypes.c_int(0)
     if emit_gain is not None:
-        if kind != EPI_RESIDUAL or emit_gain.dtype != torch.float32 or emit_gain.numel() != n:
-            raise KernelError("the next norm's rows come from the residual epilogue, with a float32 gain of the output's width")
-        emit_rows = torch.empty((batch, n), dtype=torch.bfloat16, device=x.device)
+        emit_rows = _emitted_rows(kind, emit_gain, emit_rows, batch, n, x.device)
         emit_ssq = torch.empty((8 * -(-n // 128), SSQ_COLUMNS), dtype=torch.float32, device=x.device)
     ssq, count, _, width, eps = _norm_args(norm_parts, batch, SSQ_COLUMNS)
     lib = wide_gemm_lib()
     _run(lib, lib.mb_wide_gemm(_p(x), x.stride(0), _p(weight), weight.stride(0), _p(out), out.stride(0), batch, n_w, k,
                                epilogue, _sm_count(x.device), ssq, count, width, eps, _p(emit_gain), _p(emit_rows),
-                               emit_rows.stride(0) if emit_rows is not None else 0, _p(emit_ssq), ctypes.byref(written), _stream()))
+                               emit_rows.stride(0) if emit_rows is not None else 0, _p(emit_ssq), ctypes.byref(written),
+                               _clamp_args(epilogue, clamp), _stream()))
     if emit_gain is not None:
         return out, emit_rows, emit_ssq, written.value
     return out
@@ -1921,16 +1979,16 @@ def wide_qkv_rope(x: torch.Tensor, weight: torch.Tensor, heads: int, kv_heads: i
 
 
 def tensor_core_gemm(a: torch.Tensor, weight: torch.Tensor, epilogue: int = EPI_BF16, out: Optional[torch.Tensor] = None,
-                     norm_parts=None, emit_gain: Optional[torch.Tensor] = None):
+                     norm_parts=None, emit_gain: Optional[torch.Tensor] = None, emit_rows: Optional[torch.Tensor] = None, clamp=None):
     """The tcgen05 product for this many rows: up to 128 the wide decode form, above the prefill form.  The norms
     around a product ride in the wide form only (`norm_parts`, `emit_gain`, see wide_gemm): over a whole prompt a
     norm kernel runs at the speed of memory, and a residual epilogue that does its work, one tile per block with
     nothing to hide behind, was measured to cost as much (4 us each at 2,048 rows of 2,048)."""
     if a.shape[0] <= WIDE_ROWS:
-        return wide_gemm(a, weight, epilogue, out, norm_parts=norm_parts, emit_gain=emit_gain)
+        return wide_gemm(a, weight, epilogue, out, norm_parts=norm_parts, emit_gain=emit_gain, emit_rows=emit_rows, clamp=clamp)
     if norm_parts is not None or emit_gain is not None:
         raise KernelError("the norms ride in the products of up to 128 rows only")
-    return gemm_tcgen05(a, weight, epilogue, out)
+    return gemm_tcgen05(a, weight, epilogue, out, clamp=clamp)
 
 
 def prefill_attention_tcgen05_status(head_dim: int) -> int:
