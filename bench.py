@@ -1199,6 +1199,150 @@ def mabivik_kernels(z, peak, prompt=2048, batch=8, context=1536):
     return out
 
 
+# --design rulunex: the Rulunex decoder (one norm per layer feeding, side by side, a latent attention or a windowed attention whose
+# values are its projected keys, and a clamped gated feed-forward; a span of layers that runs twice, its passes begun by joining the
+# stream with the embedding's rows) beside a Kabanex of equal size: the package's other design of one norm and parallel sublayers.
+# Equal size: as many Kabanex layers as the Rulunex has layer runs, each with as many parameters as a run uses on average.
+
+RULUNEX_SIZES = {
+    # width, layers (RULUNEX_ORDER in turn), the looped span and how often it runs, the windowed attention's heads, key/value heads, head
+    # size, rotated part and window, the latent attention's heads, key size, rotated size, value size and rank, ff
+    "s": dict(width=1024, layers=6, loop=(2, 4, 2), heads=8, kv_heads=2, head_dim=128, rot_dims=64, window=512, latent_heads=8, dim=64,
+              rot_dim=64, vdim=128, kv_rank=256, ff=2048),
+    "m": dict(width=2048, layers=12, loop=(4, 8, 2), heads=16, kv_heads=4, head_dim=128, rot_dims=64, window=1024, latent_heads=16, dim=64,
+              rot_dim=64, vdim=128, kv_rank=256, ff=4096),
+}
+RULUNEX_ORDER = ("attention", "latent_attention")
+
+
+def rulunex_runs(z):
+    start, stop, times = z["loop"]
+    return list(range(start)) + list(range(start, stop)) * times + list(range(stop, z["layers"]))
+
+
+def rulunex_config(z):
+    mixers = {"attention": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["head_dim"], "vdim": z["head_dim"],
+                            "scale": z["head_dim"] ** -0.5, "mask": {"size": z["window"]},
+                            "rot": {"dims": z["rot_dims"], "base": 500000.0,
+                                    "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}},
+              "latent_attention": {"heads": z["latent_heads"], "dim": z["dim"], "rot_dim": z["rot_dim"], "vdim": z["vdim"], "kv_rank": z["kv_rank"],
+                                   "scale": (z["dim"] + z["rot_dim"]) ** -0.5, "rot": {"dims": z["rot_dim"], "base": 500000.0}}}
+    layers = [{"type": kind, "mixer": mixers[kind], "mlp": {"kind": "dense", "ff": z["ff"], "limit": 7.0}}
+              for kind in (RULUNEX_ORDER[i % 2] for i in range(z["layers"]))]
+    return {"architecture": "Rulunex", "vocab": DESIGN_VOCAB, "width": z["width"], "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "loop": dict(zip(("start", "stop", "times"), z["loop"])), "layers": layers}
+
+
+def rulunex_layer_params(z):
+    """Matrix parameters a layer run uses, averaged over the runs (a pass's join counted among them)."""
+    w, h, g, d = z["width"], z["heads"], z["kv_heads"], z["head_dim"]
+    lh, ld, r, v, k = z["latent_heads"], z["dim"], z["rot_dim"], z["vdim"], z["kv_rank"]
+    mixers = (w * (h + g) * d + h * d * w, w * (lh * (ld + r) + k + r + lh) + lh * (ld + v) * k + lh * v * w)
+    runs = rulunex_runs(z)
+    return (sum(mixers[i % 2] for i in runs) + z["loop"][2] * 2 * w * w) // len(runs) + 3 * w * z["ff"]
+
+
+def kabanex_of_equal_size(z):
+    """A Kabanex of the bench's size with the same width, a layer per run, and the feed-forward width (a multiple of 256) that makes
+    a layer's parameters equal."""
+    zk = dict(next(r for r in DESIGN_SIZES.values() if r["width"] == z["width"]), layers=len(rulunex_runs(z)), ff=0)
+    zk["ff"] = max(256, round((rulunex_layer_params(z) - kabanex_layer_params(zk)) / (2 * z["width"]) / 256) * 256)
+    return kabanex_config(zk)
+
+
+def rulunex_kernels(z, peak, prompt=2048, batch=8, context=1536):
+    """The design's kernels alone beside the like kernels of the other models at equal sizes, each with its fraction of the
+    measured peak that bounds it."""
+    import torch
+
+    from models_b200.kernels import ops
+    from models_b200.parts.linear import linear
+
+    dev, bf = "cuda", torch.bfloat16
+    W, F, window, page = z["width"], z["ff"], z["window"], 64
+    H, G, D = z["heads"], z["kv_heads"], z["head_dim"]
+    LH, LD, R, DV, K = (z[k] for k in ("latent_heads", "dim", "rot_dim", "vdim", "kv_rank"))
+    out = {}
+
+    def rated(us, flops=None, moved=None):
+        if flops is not None:
+            return {"us": us, "tflops": flops / us / 1e6, "frac_of_bf16_peak": flops / us / 1e6 / peak["bf16_tflops"]}
+        return {"us": us, "gbs": moved / us / 1e3, "frac_of_hbm_peak": moved / us / 1e3 / peak["hbm_gbs"]}
+
+    rnd = lambda *shape: torch.randn(shape, device=dev)  # noqa: E731
+    low = lambda *shape: rnd(*shape).to(bf)  # noqa: E731
+    longest = max(prompt, context)
+    angle = torch.arange(longest, dtype=torch.float32, device=dev)[:, None]
+    tables = lambda pairs: tuple(f(angle * torch.rand((1, pairs), device=dev)).contiguous() for f in (torch.cos, torch.sin))  # noqa: E731
+    cos, sin = tables(R // 2)
+    cos_a, sin_a = tables(z["rot_dims"] // 2)
+    for name, rows, cu_q, lengths, q_len in (("prompt", prompt, [0, prompt], [prompt], prompt),
+                                             ("decode", batch, list(range(batch + 1)), [context] * batch, 1)):
+        sequences = len(lengths)
+        cu = torch.tensor(cu_q, dtype=torch.int32, device=dev)
+        kv = torch.tensor(lengths, dtype=torch.int32, device=dev)
+        count = lambda rule: sum(rule(p) for n in lengths for p in range(n - q_len, n))  # noqa: E731  (query, key) pairs of a head
+        windowed, chunked, all_pairs = count(lambda p: min(p + 1, window)), count(lambda p: p % window + 1), count(lambda p: p + 1)
+        positions = torch.cat([torch.arange(n - q_len, n) for n in lengths]).to(torch.int32).to(dev)
+        pages = sequences * (-(-lengths[0] // page))
+        table = (torch.arange(pages, dtype=torch.int32, device=dev) + 1).reshape(sequences, -1).contiguous()
+        mapping = (torch.arange(rows, dtype=torch.int32, device=dev) + page)
+        # latent attention over every earlier position, a gate per head; beside Mabivik's (a window, a query latent, gates per element)
+        pool = low(pages + 1, 1, page, K + R)
+        q, o = low(rows, LH * (K + R)), torch.empty((rows, LH * K), dtype=bf, device=dev)
+        for title, win, used in (("latent_attention", 0, all_pairs), ("latent_attention_mabivik", window, windowed)):
+            us = time_kernel(lambda: ops.gated_attention(q, o, pool, None, table, cu, kv, q_len, LH, 1, K + R, K, "softmax", LD ** -0.5, window=win))
+            out[f"{name}_{title}"] = rated(us, flops=used * LH * (2 * (K + R) + 2 * K)) if q_len > 1 else \
+                rated(us, moved=sum(min(n, win or n) for n in lengths) * (K + R) * 2)
+        x, y = low(rows, LH * (LD + R)), torch.empty((rows, LH * DV), dtype=bf, device=dev)
+        into, outof = low(LH, K, LD), low(LH, DV, K)
+        for title, gate, kind in (("head_products", low(rows, LH), "head"), ("head_products_mabivik", low(rows, LH * DV), "element")):
+            us = time_kernel(lambda: (ops.head_linear(x, into, q, LH, turned=R, cos=cos, sin=sin, positions=positions),
+                                      ops.head_linear(o, outof, y, LH, gate, gate_kind=kind)))
+            out[f"{name}_{title}"] = rated(us, flops=rows * LH * 2 * K * (LD + DV)) if q_len > 1 else \
+                rated(us, moved=LH * K * (LD + DV) * 2 + rows * LH * (LD + K + K + DV) * 2)
+        Q = K * 2
+        first, gq, gk = low(rows, Q + K + R), torch.ones(Q, device=dev), torch.ones(K, device=dev)
+        us = time_kernel(lambda: ops.latent_prepare(None, None, 0, first[:, Q:], gk, R, cos, sin, positions, 1e-6, pool, mapping))
+        out[f"{name}_latent_prepare"] = rated(us, moved=rows * 4 * (K + R))
+        us = time_kernel(lambda: ops.latent_prepare(first[:, :Q], gq, Q, first[:, Q:], gk, R, cos, sin, positions, 1e-6, pool, mapping))
+        out[f"{name}_latent_prepare_mabivik"] = rated(us, moved=rows * 4 * (Q + K + R))
+        # windowed attention with the projected keys as values; beside Rolevik's over chunks as long as the window, values of their own
+        k_pool, v_pool = low(pages + 1, G, page, D), low(pages + 1, G, page, D)
+        aq, ao = low(rows, H * D), torch.empty((rows, H * D), dtype=bf, device=dev)
+        for title, more, used in (("attention", {"window": window}, windowed), ("attention_rolevik", {"block": window}, chunked)):
+            us = time_kernel(lambda: ops.gated_attention(aq, ao, k_pool, v_pool, table, cu, kv, q_len, H, G, D, D, "softmax", D ** -0.5, **more))
+            out[f"{name}_{title}"] = rated(us, flops=used * H * 4 * D) if q_len > 1 else rated(us, moved=used * G * 2 * D * 2)
+        proj = low(rows, (H + 2 * G) * D)
+        aq, ak, av = proj[:, :H * D], proj[:, H * D:(H + G) * D], proj[:, (H + G) * D:]
+        qg, kg = torch.ones(H * D, device=dev), torch.ones(G * D, device=dev)
+        for title, v, parts in (("project_norm_rotate_store", ak, 2 * H + 3 * G), ("project_norm_rotate_store_rolevik", av, 2 * H + 4 * G)):
+            us = time_kernel(lambda: ops.project_norm_rotate_store(aq, ak, v, None, None, None, qg, kg, 1e-6, positions, cos_a, sin_a, z["rot_dims"],
+                                                                   False, k_pool, v_pool, mapping, H, G, D, D))
+            out[f"{name}_{title}"] = rated(us, moved=rows * parts * D * 2)
+        # the layer's first product with the gate/up pairs in its epilogue; beside Llama's norm, q/k/v rows and silu pairs
+        plain = LH * (LD + R) + K + R + LH
+        w_in = (rnd(plain + 2 * F, W) * 0.02).to(bf)
+        stream, gain = rnd(rows, W), torch.ones(W, device=dev)
+        h, mid, clamp = low(rows, W), torch.empty((rows, F), dtype=bf, device=dev), (7.0, 1.702, 1.0)
+        if q_len > 1:
+            us = time_kernel(lambda: (ops.tensor_core_gemm(h, w_in[plain:], ops.EPI_CLAMPED, out=mid, clamp=clamp), ops.tensor_core_gemm(h, w_in[:plain])))
+            us2 = time_kernel(lambda: (ops.tensor_core_gemm(h, w_in[plain:], ops.EPI_SWIGLU, out=mid), ops.tensor_core_gemm(h, w_in[:plain])))
+        else:
+            us = time_kernel(lambda: ops.skinny_gemm_pairs(w_in, plain, mid, clamp, xf=stream, gain=gain, eps=1e-6))
+            us2 = time_kernel(lambda: (ops.skinny_gemm(w_in[plain:], ops.EPI_SWIGLU, xf=stream, gain=gain, eps=1e-6),
+                                       ops.skinny_gemm(w_in[:plain], ops.EPI_BF16, xf=stream, gain=gain, eps=1e-6)))
+        work = {"flops": 2 * rows * W * (plain + 2 * F)} if q_len > 1 else {"moved": (plain + 2 * F) * W * 2}
+        out[f"{name}_first_product"], out[f"{name}_first_product_llama"] = rated(us, **work), rated(us2, **work)
+        # the join ahead of a pass; beside a plain product of the same sizes
+        w_join, both = (rnd(W, 2 * W) * 0.02).to(bf), torch.empty((rows, 2 * W), dtype=bf, device=dev)
+        work = {"flops": 4 * rows * W * W} if q_len > 1 else {"moved": 4 * W * W}
+        us = time_kernel(lambda: (ops.store_columns(stream, both[:, :W]), linear(both, w_join, torch.float32)))
+        out[f"{name}_join"] = rated(us, **work)
+        out[f"{name}_join_product_alone"] = rated(time_kernel(lambda: linear(both, w_join, torch.float32)), **work)
+    return out
+
+
 def design_run(args) -> int:
     import torch
 
@@ -1220,6 +1364,10 @@ def design_run(args) -> int:
         title, all_sizes, make, params, beside, alone = "Mabivik", MABIVIK_SIZES, mabivik_config, mabivik_layer_params, \
             rolevik_of_equal_size, mabivik_kernels
         other, other_title = "rolevik", "Rolevik of equal size (the parameters a token uses)"
+    elif args.design == "rulunex":
+        title, all_sizes, make, params, beside, alone = "Rulunex", RULUNEX_SIZES, rulunex_config, rulunex_layer_params, \
+            kabanex_of_equal_size, rulunex_kernels
+        other, other_title = "kabanex", "Kabanex of equal size (a layer per layer run, the parameters a run uses)"
     else:
         title, all_sizes, make, params, beside, alone = "Lovurax", LOVURAX_SIZES, lovurax_config, lovurax_layer_params, \
             (lambda z: llama_of_equal_size(z, lovurax_layer_params(z))), lovurax_kernels
@@ -1268,8 +1416,8 @@ def main() -> int:
     parser.add_argument("--only-prefill", action="store_true",
                         help="run the workload's prefill alone and print its figures (for profiling)")
     parser.add_argument("--size", default=None, choices=["s", "m"], help="with --design: one of its two sizes alone")
-    parser.add_argument("--design", default=None, choices=["kabanex", "lovurax", "kivezen", "rolevik", "mabivik"],
-                        help="instead of the default run: this design beside a model of equal size (a Llama; for kivezen a Lovurax, for rolevik a Kivezen, for mabivik a Rolevik): "
+    parser.add_argument("--design", default=None, choices=["kabanex", "lovurax", "kivezen", "rolevik", "mabivik", "rulunex"],
+                        help="instead of the default run: this design beside a model of equal size (a Llama; for kivezen a Lovurax, for rolevik a Kivezen, for mabivik a Rolevik, for rulunex a Kabanex): "
                              "prefill, decode, its kernels alone")
     args = parser.parse_args()
     if args.design and args.impl == "ours":

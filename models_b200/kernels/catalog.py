@@ -24,6 +24,7 @@ LIBRARIES = [
     ("mb_gated_attention_tc", ["gated_attention_tc.cu"], {"MB_KEY_DIM": 64, "MB_VALUE_DIM": 128, "MB_SHARED_ROWS": 0}),
     ("mb_gated_attention_tc", ["gated_attention_tc.cu"], {"MB_KEY_DIM": 256, "MB_VALUE_DIM": 256, "MB_SHARED_ROWS": 1}),
     ("mb_gated_attention_tc", ["gated_attention_tc.cu"], {"MB_KEY_DIM": 320, "MB_VALUE_DIM": 256, "MB_SHARED_ROWS": 1}),
+    ("mb_gated_attention_tc", ["gated_attention_tc.cu"], {"MB_KEY_DIM": 128, "MB_VALUE_DIM": 128, "MB_SHARED_ROWS": 0}),
     # the state-space chunks are compiled per size of a head's state; these are the sizes of the benchmark's models of that design
     ("mb_state_space_chunks", ["state_space_chunks.cu"], {"MB_STATE": 128, "MB_VALUE_DIM": 64}),
     ("mb_random_init", ["random_init.cu"], {}),
