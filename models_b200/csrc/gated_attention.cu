@@ -345,6 +345,233 @@ __global__ void project_norm_rotate_store_kernel(T* __restrict__ q, int q_stride
     }
 }
 
+// The same on whole rows of 8 elements a thread: head_dim, value_dim and half of the rotated part multiples of 8 (interleaved pairs: the
+// rotated part), rows on 16 bytes (float: 32).  grid (tokens); shared memory: a row of q and one of k as floats.
+template <typename T>
+__global__ void project_norm_rotate_store_vec8_kernel(T* __restrict__ q, int q_stride, const T* __restrict__ k, int k_stride,
+                                                      const T* __restrict__ v, int v_stride, const float* __restrict__ q_bias,
+                                                      const float* __restrict__ k_bias, const float* __restrict__ v_bias,
+                                                      const float* __restrict__ q_gain, const float* __restrict__ k_gain, float eps,
+                                                      const int* __restrict__ positions, Rotation rotation, T* __restrict__ k_pool,
+                                                      T* __restrict__ v_pool, const int* __restrict__ slot_mapping, int heads, int kv_heads,
+                                                      int head_dim, int value_dim, int page_size) {
+    grid_launch_dependents();
+    __shared__ float2 scratch[32];
+    extern __shared__ __align__(16) float both_rows[];
+    const int token = blockIdx.x;
+    const int q_width = heads * head_dim, k_width = kv_heads * head_dim;
+    const int q_chunks = q_width / 8, chunks = q_chunks + k_width / 8;
+    // (positions and slots are written before the step begins)
+    const int pos = positions[token], slot = slot_mapping[token];
+    const size_t page = slot >= 0 ? slot / page_size : 0, offset = slot >= 0 ? slot % page_size : 0;
+    grid_dependency_wait();
+    float2 squares = make_float2(0.0f, 0.0f);
+    for (int c = threadIdx.x; c < chunks; c += blockDim.x) {
+        const bool is_query = c < q_chunks;
+        const int at = (is_query ? c : c - q_chunks) * 8;
+        float x[8];
+        load8(is_query ? q + (size_t)token * q_stride + at : k + (size_t)token * k_stride + at, x);
+        const float* bias = is_query ? q_bias : k_bias;
+        if (bias != nullptr) {
+            float b[8];
+            load8(bias + at, b);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) x[j] += b[j];
+        }
+        store8(both_rows + c * 8, x);
+        float sum = 0.0f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) sum = fmaf(x[j], x[j], sum);
+        if (is_query) squares.x += sum;
+        else squares.y += sum;
+    }
+    // both rows' sums at once: warps by shuffles, then the warps in their order
+    squares.x = warp_sum(squares.x);
+    squares.y = warp_sum(squares.y);
+    if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = squares;
+    __syncthreads();
+    float2 total = make_float2(0.0f, 0.0f);
+    for (int w = 0; w < (int)(blockDim.x + 31) / 32; ++w) {
+        total.x += scratch[w].x;
+        total.y += scratch[w].y;
+    }
+    const float q_factor = q_gain != nullptr ? 1.0f / sqrtf(total.x / (float)q_width + eps) : 1.0f;
+    const float k_factor = k_gain != nullptr ? 1.0f / sqrtf(total.y / (float)k_width + eps) : 1.0f;
+    const int turning = rotation.dim, half = turning / 2;
+    for (int c = threadIdx.x; c < chunks; c += blockDim.x) {
+        const bool is_query = c < q_chunks;
+        if (!is_query && slot < 0) continue;
+        const int at = (is_query ? c : c - q_chunks) * 8;
+        const int head = at / head_dim, d = at % head_dim;
+        const float* row = is_query ? both_rows : both_rows + q_width;
+        const float* gain = is_query ? q_gain : k_gain;
+        const float factor = is_query ? q_factor : k_factor;
+        float x[8], g[8];
+        load8(row + at, x);
+        if (gain != nullptr) {
+            load8(gain + at, g);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) x[j] = x[j] * factor * g[j];
+        }
+        if (d < turning && !rotation.interleaved) {
+            const bool first = d < half;
+            const int other = first ? at + half : at - half, pair = first ? d : d - half;
+            float y[8], cs[8], sn[8];
+            load8(row + other, y);
+            if (gain != nullptr) {
+                load8(gain + other, g);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) y[j] = y[j] * factor * g[j];
+            }
+            load8(rotation.cos + (size_t)pos * half + pair, cs);
+            load8(rotation.sin + (size_t)pos * half + pair, sn);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) x[j] = first ? x[j] * cs[j] - y[j] * sn[j] : x[j] * cs[j] + y[j] * sn[j];
+        } else if (d < turning) {
+#pragma unroll
+            for (int j = 0; j < 8; j += 2) {
+                const float cs = rotation.cos[(size_t)pos * half + (d + j) / 2], sn = rotation.sin[(size_t)pos * half + (d + j) / 2];
+                const float u = x[j], w = x[j + 1];
+                x[j] = u * cs - w * sn;
+                x[j + 1] = w * cs + u * sn;
+            }
+        }
+        store8(is_query ? q + (size_t)token * q_stride + at : k_pool + ((page * kv_heads + head) * page_size + offset) * head_dim + d, x);
+    }
+    if (slot < 0 || value_dim <= 0) return;
+    for (int c = threadIdx.x; c < kv_heads * value_dim / 8; c += blockDim.x) {
+        const int at = c * 8, head = at / value_dim, d = at % value_dim;
+        float x[8];
+        load8(v + (size_t)token * v_stride + at, x);
+        if (v_bias != nullptr) {
+            float b[8];
+            load8(v_bias + at, b);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) x[j] += b[j];
+        }
+        store8(v_pool + ((page * kv_heads + head) * page_size + offset) * value_dim + d, x);
+    }
+}
+
+// What a latent attention without a query latent does to its first product's rows.  grid (tokens); block 128: warp 0 makes the cached row
+// [latent | tail] -- the latent divided by its root mean square, times its gain; the tail's `turned` numbers rotated by the token's
+// position (pairs (i, i + turned / 2), tables [positions][turned / 2]) -- into the pool at the token's slot.  For a prompt that reads
+// its own rows (prompt.latent given) the row is also left in the step's order, [tokens][latent] and [tokens][padded] with zeros behind
+// the tail, and the other warps rotate the query heads' tails into [tokens][heads * padded].
+struct PromptRows {
+    void* latent;         // [tokens][latent]
+    void* tail;           // [tokens][padded], null where there is no tail
+    const void* q;        // query rows: head h's tail at column h * (q_head + turned) + q_head
+    int q_stride, q_head, heads;
+    void* q_tail;         // [tokens][heads * padded]
+    int padded;
+};
+
+template <typename T, bool kVector>
+__global__ void __launch_bounds__(128)
+latent_rows_kernel(const T* __restrict__ k, int k_stride, const float* __restrict__ gain, int latent, int turned, const float* __restrict__ cos,
+                   const float* __restrict__ sin, const int* __restrict__ positions, float eps, T* __restrict__ k_pool,
+                   const int* __restrict__ slot_mapping, PromptRows prompt) {
+    grid_launch_dependents();
+    const size_t token = blockIdx.x;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = turned / 2;
+    const float* cos_row = nullptr;
+    const float* sin_row = nullptr;
+    if (turned > 0) {
+        const size_t pos = positions[token];
+        cos_row = cos + pos * half;
+        sin_row = sin + pos * half;
+    }
+    const int slot = warp == 0 ? slot_mapping[token] : -1;
+    grid_dependency_wait();
+    if (warp == 0) {
+        if (slot < 0 && prompt.latent == nullptr) return;
+        const T* src = k + token * k_stride;
+        T* row = slot >= 0 ? k_pool + (size_t)slot * (latent + turned) : nullptr;  // [page][1][page_size][latent + turned]: the slot counts rows
+        T* own = prompt.latent != nullptr ? (T*)prompt.latent + token * latent : nullptr;
+        T* own_tail = prompt.latent != nullptr && turned > 0 ? (T*)prompt.tail + token * prompt.padded : nullptr;
+        float squares = 0.0f;
+        if (kVector) {
+            for (int i = lane * 8; i < latent; i += 256) {
+                float x[8];
+                load8(src + i, x);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) squares = fmaf(x[j], x[j], squares);
+            }
+        } else {
+            for (int i = lane; i < latent; i += 32) {
+                const float x = Num<T>::load(src + i);
+                squares = fmaf(x, x, squares);
+            }
+        }
+        const float factor = 1.0f / sqrtf(warp_sum(squares) / (float)latent + eps);
+        if (kVector) {
+            for (int i = lane * 8; i < latent; i += 256) {
+                float x[8], g[8];
+                load8(src + i, x);
+                load8(gain + i, g);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) x[j] = x[j] * factor * g[j];
+                if (row != nullptr) store8(row + i, x);
+                if (own != nullptr) store8(own + i, x);
+            }
+        } else {
+            for (int i = lane; i < latent; i += 32) {
+                const float x = Num<T>::load(src + i) * factor * gain[i];
+                if (row != nullptr) Num<T>::store(row + i, x);
+                if (own != nullptr) Num<T>::store(own + i, x);
+            }
+        }
+        for (int i = lane; i < half; i += 32) {
+            const float u = Num<T>::load(src + latent + i), w = Num<T>::load(src + latent + half + i);
+            const float a = u * cos_row[i] - w * sin_row[i], b = w * cos_row[i] + u * sin_row[i];
+            if (row != nullptr) {
+                Num<T>::store(row + latent + i, a);
+                Num<T>::store(row + latent + half + i, b);
+            }
+            if (own_tail != nullptr) {
+                Num<T>::store(own_tail + i, a);
+                Num<T>::store(own_tail + half + i, b);
+            }
+        }
+        if (own_tail != nullptr)
+            for (int i = turned + lane; i < prompt.padded; i += 32) Num<T>::store(own_tail + i, 0.0f);
+        return;
+    }
+    if (prompt.latent == nullptr || turned <= 0) return;
+    const T* q_row = (const T*)prompt.q + token * prompt.q_stride + prompt.q_head;
+    T* out_row = (T*)prompt.q_tail + token * prompt.heads * prompt.padded;
+    const int mine = threadIdx.x - 32, head_columns = prompt.q_head + turned;
+    if (kVector && half % 8 == 0) {
+        const int per_head = half / 8;
+        for (int c = mine; c < prompt.heads * per_head; c += 96) {
+            const int head = c / per_head, i = (c % per_head) * 8;
+            float u[8], w[8], cs[8], sn[8];
+            load8(q_row + (size_t)head * head_columns + i, u);
+            load8(q_row + (size_t)head * head_columns + half + i, w);
+            load8(cos_row + i, cs);
+            load8(sin_row + i, sn);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                const float a = u[j] * cs[j] - w[j] * sn[j];
+                w[j] = w[j] * cs[j] + u[j] * sn[j];
+                u[j] = a;
+            }
+            store8(out_row + (size_t)head * prompt.padded + i, u);
+            store8(out_row + (size_t)head * prompt.padded + half + i, w);
+        }
+    } else {
+        for (int c = mine; c < prompt.heads * half; c += 96) {
+            const int head = c / half, i = c % half;
+            const float u = Num<T>::load(q_row + (size_t)head * head_columns + i), w = Num<T>::load(q_row + (size_t)head * head_columns + half + i);
+            Num<T>::store(out_row + (size_t)head * prompt.padded + i, u * cos_row[i] - w * sin_row[i]);
+            Num<T>::store(out_row + (size_t)head * prompt.padded + half + i, w * cos_row[i] + u * sin_row[i]);
+        }
+    }
+    const int zeros = prompt.padded - turned;
+    for (int c = mine; c < prompt.heads * zeros; c += 96) Num<T>::store(out_row + (size_t)(c / zeros) * prompt.padded + turned + c % zeros, 0.0f);
+}
+
 // grid (tokens, 2); block 128 (block 0 of a token: the query's latent; block 1: the cached row).  What a latent attention does to
 // the rows of its first product: the query's latent (q_width numbers,
 // null: none) divided by its root mean square and multiplied by its gain, into rows of its own that are zero up to q_columns;
@@ -1351,6 +1578,24 @@ MB_EXPORT int mb_project_norm_rotate_store(void* q, int q_stride, const void* k,
     const size_t smem = sizeof(float) * (size_t)(heads + kv_heads) * head_dim;
     if (smem > 40 * 1024) return fail("project_norm_rotate_store: rows of %d numbers exceed the 10240 a block keeps", (heads + kv_heads) * head_dim);
     const Rotation rotation{cos, sin, rotary_dim, interleaved, 0, nullptr, nullptr, 0};
+    const size_t element = dtype == MB_F32 ? 4 : 2, row_bytes = 8 * element - 1;
+    const bool wide = head_dim % 8 == 0 && value_dim % 8 == 0 && rotary_dim % (interleaved ? 8 : 16) == 0 && q_stride % 8 == 0 && k_stride % 8 == 0 &&
+                      v_stride % 8 == 0 && !(((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)k_pool | (uintptr_t)v_pool) & row_bytes) &&
+                      !(((uintptr_t)q_bias | (uintptr_t)k_bias | (uintptr_t)v_bias | (uintptr_t)q_gain | (uintptr_t)k_gain | (uintptr_t)cos | (uintptr_t)sin) & 15);
+    if (wide && (dtype == MB_F32 || dtype == MB_BF16)) {
+        const int chunks = (heads + kv_heads) * head_dim / 8;
+        const int block = chunks >= 512 ? 512 : (chunks + 31) / 32 * 32;
+        if (dtype == MB_F32)
+            MB_LAUNCH("project_norm_rotate_store", project_norm_rotate_store_vec8_kernel<float>, dim3(tokens), dim3(block), smem, stream, true,
+                      (float*)q, q_stride, (const float*)k, k_stride, (const float*)v, v_stride, q_bias, k_bias, v_bias, q_gain, k_gain, eps,
+                      positions, rotation, (float*)k_pool, (float*)v_pool, slot_mapping, heads, kv_heads, head_dim, value_dim, page_size);
+        else
+            MB_LAUNCH("project_norm_rotate_store", project_norm_rotate_store_vec8_kernel<__nv_bfloat16>, dim3(tokens), dim3(block), smem, stream,
+                      true, (__nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)k, k_stride, (const __nv_bfloat16*)v, v_stride, q_bias, k_bias,
+                      v_bias, q_gain, k_gain, eps, positions, rotation, (__nv_bfloat16*)k_pool, (__nv_bfloat16*)v_pool, slot_mapping, heads,
+                      kv_heads, head_dim, value_dim, page_size);
+        return check_launch("project_norm_rotate_store");
+    }
     const int threads = (heads + kv_heads) * head_dim >= 1024 ? 256 : 128;
     if (dtype == MB_F32)
         MB_LAUNCH("project_norm_rotate_store", project_norm_rotate_store_kernel<float>, dim3(tokens), dim3(threads), smem, stream, true,
@@ -1386,6 +1631,41 @@ MB_EXPORT int mb_latent_prepare(const void* q, int q_stride, const float* q_gain
     else
         return fail("latent_prepare: unknown dtype code %d", dtype);
     return check_launch("latent_prepare");
+}
+
+template <typename T>
+static int launch_latent_rows(const void* k, int k_stride, const float* gain, int latent, int turned, const float* cos, const float* sin,
+                              const int* positions, float eps, void* k_pool, const int* slot_mapping, const PromptRows& prompt, int tokens,
+                              cudaStream_t stream) {
+    const size_t row_bytes = 8 * sizeof(T) - 1;
+    const bool wide = latent % 8 == 0 && turned % 8 == 0 && k_stride % 8 == 0 && prompt.padded % 8 == 0 && prompt.q_stride % 8 == 0 && prompt.q_head % 8 == 0 &&
+                      !(((uintptr_t)k | (uintptr_t)k_pool | (uintptr_t)prompt.latent | (uintptr_t)prompt.q | (uintptr_t)prompt.q_tail) & row_bytes) &&
+                      !(((uintptr_t)gain | (uintptr_t)cos | (uintptr_t)sin) & 15);
+    const dim3 block(prompt.latent != nullptr && turned > 0 ? 128 : 32);
+    if (wide)
+        MB_LAUNCH("latent_rows", (latent_rows_kernel<T, true>), dim3(tokens), block, 0, stream, true, (const T*)k, k_stride, gain, latent, turned,
+                  cos, sin, positions, eps, (T*)k_pool, slot_mapping, prompt);
+    else
+        MB_LAUNCH("latent_rows", (latent_rows_kernel<T, false>), dim3(tokens), block, 0, stream, true, (const T*)k, k_stride, gain, latent, turned,
+                  cos, sin, positions, eps, (T*)k_pool, slot_mapping, prompt);
+    return check_launch("latent_rows");
+}
+
+// k: rows [latent | tail] of one storage type (stride in elements); see latent_rows_kernel.  own_latent null: nothing but the pool's row is
+// made; else own_latent [tokens][latent], own_tail [tokens][padded], q (heads of q_head + turned columns) and q_tail [tokens][heads * padded].
+MB_EXPORT int mb_latent_rows(const void* k, int k_stride, const float* gain, int latent, int turned, const float* cos, const float* sin,
+                             const int* positions, float eps, void* k_pool, const int* slot_mapping, void* own_latent, void* own_tail,
+                             const void* q, int q_stride, int q_head, int heads, void* q_tail, int padded, int dtype, int tokens,
+                             cudaStream_t stream) {
+    if (tokens <= 0) return 0;
+    if (latent <= 0 || turned < 0 || turned % 2 || (turned > 0 && (cos == nullptr || sin == nullptr))) return fail("latent_rows: rows of %d and %d numbers", latent, turned);
+    if (own_latent != nullptr && turned > 0 && (!own_tail || !q || !q_tail || padded < turned || heads <= 0))
+        return fail("latent_rows: a prompt's tails of %d numbers in %d columns need their tensors", turned, padded);
+    const PromptRows prompt{own_latent, own_tail, q, q_stride, q_head, heads, q_tail, padded};
+    if (dtype == MB_F32) return launch_latent_rows<float>(k, k_stride, gain, latent, turned, cos, sin, positions, eps, k_pool, slot_mapping, prompt, tokens, stream);
+    if (dtype == MB_BF16)
+        return launch_latent_rows<__nv_bfloat16>(k, k_stride, gain, latent, turned, cos, sin, positions, eps, k_pool, slot_mapping, prompt, tokens, stream);
+    return fail("latent_rows: unknown dtype code %d", dtype);
 }
 
 // The second half of mb_gated_attention_decode alone: adds the runs that another kernel left in `partial` (bfloat16 results, softmax).

@@ -39,6 +39,7 @@ class StepBatch:
     max_kv_len: int
     q_lens: Tuple[int, ...]  # host copies, for parts that loop on the host
     host_slots: Tuple[int, ...]
+    fresh: bool = False  # every sequence of the step starts with it: all the keys its tokens see are the step's own
 
 
 @dataclass(frozen=True)
@@ -131,7 +132,7 @@ def pack_step(cache, entries, layout: StepLayout, buf: np.ndarray, state_pad_row
     return q_lens, max_kv
 
 
-def batch_from_buffer(dev: torch.Tensor, layout: StepLayout, q_lens, max_kv: int, host_slots) -> StepBatch:
+def batch_from_buffer(dev: torch.Tensor, layout: StepLayout, q_lens, max_kv: int, host_slots, fresh: bool = False) -> StepBatch:
     offsets = layout.offsets
     part = [dev[int(offsets[i]):int(offsets[i + 1])] for i in range(len(layout.sizes))]
     B, width = layout.sequences, layout.blocks
@@ -140,7 +141,12 @@ def batch_from_buffer(dev: torch.Tensor, layout: StepLayout, q_lens, max_kv: int
         tokens=part[0], positions=part[1], cu_q=part[2], kv_lens=part[3], slots=part[4],
         want_rows=part[5] if layout.wanted else None, groups=groups, num_sequences=B, num_tokens=layout.tokens,
         num_wanted=layout.wanted, max_q_len=max(q_lens), max_kv_len=max_kv, q_lens=tuple(q_lens),
-        host_slots=tuple(host_slots))
+        host_slots=tuple(host_slots), fresh=fresh)
+
+
+def starts_sequences(cache, entries) -> bool:
+    """Whether no sequence of the step holds anything yet."""
+    return all(cache.lengths[slot] == 0 for slot, _, _ in entries)
 
 
 def build_step_batch(cache, entries: Sequence[Tuple[int, Sequence[int], Sequence[int]]], device,
@@ -156,4 +162,4 @@ def build_step_batch(cache, entries: Sequence[Tuple[int, Sequence[int], Sequence
         dev = host.pin_memory().to(device, non_blocking=True)
     else:
         dev = host.to(device)
-    return batch_from_buffer(dev, layout, q_lens, max_kv, [slot for slot, _, _ in entries])
+    return batch_from_buffer(dev, layout, q_lens, max_kv, [slot for slot, _, _ in entries], starts_sequences(cache, entries))

@@ -21,7 +21,7 @@ import numpy as np
 import torch
 
 from ..kernels import ops
-from .batch import StepLayout, batch_from_buffer, pack_step
+from .batch import StepLayout, batch_from_buffer, pack_step, starts_sequences
 
 
 def ladder(max_batch: int) -> List[int]:
@@ -95,7 +95,7 @@ class _Captured:
     """One captured step: `size` sequences of one token each, or with `tokens` a step of so many
     rows shared by up to `size` sequences in any way."""
 
-    def __init__(self, engine, size: int, blocks: int, pool, span: int = 0, tokens: Optional[int] = None):
+    def __init__(self, engine, size: int, blocks: int, pool, span: int = 0, tokens: Optional[int] = None, fresh: bool = False):
         self.size = size
         self.span = span  # the class of context lengths the capture is for (ops.decode_span)
         cache = engine.cache
@@ -112,7 +112,7 @@ class _Captured:
         self.dev.copy_(self.host)
         # the sizes kernels are launched with: one token each, or as if one sequence held every row
         q_lens = [tokens] + [0] * (size - 1) if prompts else [1] * size
-        self.batch = batch_from_buffer(self.dev, self.layout, q_lens, max(1, span), [])
+        self.batch = batch_from_buffer(self.dev, self.layout, q_lens, max(1, span), [], fresh)
         stream = torch.cuda.Stream(device=engine.device)
         stream.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(stream):
@@ -246,7 +246,7 @@ class PromptGraphs:
     def __init__(self, decode_graphs: DecodeGraphs):
         self.decode_graphs = decode_graphs
         self.engine = decode_graphs.engine
-        self.captured: Dict[tuple, _Captured] = {}  # (batch size, token count, page-table width)
+        self.captured: Dict[tuple, _Captured] = {}  # (batch size, token count, page-table width, whether the sequences start)
         self.uses: Dict[tuple, int] = {}
 
     def bucket(self, entries: Sequence) -> Optional[tuple]:
@@ -263,7 +263,7 @@ class PromptGraphs:
         longest = max(cache.lengths[slot] + len(tokens) for slot, tokens, _ in entries)
         if -(-longest // cache.page_size) > graphs.blocks:
             return None
-        return size, next(t for t in PROMPT_TOKENS if t >= total), graphs.table_width(longest)
+        return size, next(t for t in PROMPT_TOKENS if t >= total), graphs.table_width(longest), starts_sequences(cache, entries)
 
     def step(self, entries: Sequence) -> Optional[torch.Tensor]:
         """entries: (slot, tokens, wanted places); the cache already has room.  Returns the logits of
@@ -278,7 +278,7 @@ class PromptGraphs:
             if self.uses[key] <= EAGER_USES or len(self.captured) >= MAX_PROMPT_CAPTURES:
                 return None
             graphs = self.decode_graphs
-            captured = self.captured[key] = _Captured(self.engine, key[0], key[2], graphs.pool, tokens=key[1])
+            captured = self.captured[key] = _Captured(self.engine, key[0], key[2], graphs.pool, tokens=key[1], fresh=key[3])
         wanted = captured.fill(self.engine.cache, entries)
         captured.upload()
         captured.graph.replay()

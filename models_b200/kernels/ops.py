@@ -826,6 +826,60 @@ def gated_attention_tc_takes(q: torch.Tensor, out: torch.Tensor, k_pool: torch.T
     return gate is None or gate_kind != "element" or (gate.stride(0) % 2 == 0 and gate.data_ptr() % 4 == 0)
 
 
+def float_weight_attention_library(key_dim: int, value_dim: int, turned: int = 0, contiguous: bool = False):
+    """The tcgen05 prompt attention with float weights, compiled for these sizes (multiples of 64) at first use."""
+    return load_library("mb_prefill_attention_tcgen05", ["prefill_attention_tcgen05.cu"],
+                        {"MB_KEY_DIM": int(key_dim), "MB_VALUE_DIM": int(value_dim), "MB_TURNED_DIM": int(turned),
+                         "MB_CONTIGUOUS": 1 if contiguous else 0})
+
+
+def float_weight_attention_takes(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, v_pool: Optional[torch.Tensor], head_dim: int,
+                                 value_dim: int, max_q_len: int) -> bool:
+    """bfloat16, cache pages of 64, keys of 64, 128, 192 or 256 numbers and values of 64 or 128 of their own, steps of more than a
+    few tokens, rows that TMA and 16-byte stores can address."""
+    return (q.dtype == torch.bfloat16 and v_pool is not None and k_pool.shape[2] == 64 and head_dim % 64 == 0 and 64 <= head_dim <= 256
+            and value_dim in (64, 128) and max_q_len >= TCGEN05_ATTENTION_MIN_ROWS and q.stride(0) % 8 == 0 and out.stride(0) % 8 == 0
+            and q.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0 and k_pool.data_ptr() % 16 == 0 and v_pool.data_ptr() % 16 == 0)
+
+
+def prompt_attention(q: torch.Tensor, q_tail: Optional[torch.Tensor], k: torch.Tensor, v: torch.Tensor, k_tail: Optional[torch.Tensor],
+                     out: torch.Tensor, cu_q: torch.Tensor, kv_lens: torch.Tensor, max_q_len: int, heads: int, head_columns: int,
+                     value_columns: int, scale: float, gate: Optional[torch.Tensor] = None, window: int = 0) -> None:
+    """Causal softmax attention of prompts that start their sequences, on the tcgen05 tensor cores with float weights: every key comes
+    from the step's own rows.  bfloat16: k [T, heads * KD] and v [T, heads * VD] (column slices with one row stride; KD, VD multiples
+    of 64, heads padded with zero columns), k_tail [T, RD] shared by all heads and q_tail [T, heads * RD] (or None, None); q [T, ...] holds
+    head h's own coordinates from column h * head_columns on; out [T, heads * value_columns]; gate [T, heads]: head h's result is
+    multiplied by its sigmoid.  `window` n > 0: query i sees key j only if i - j < n."""
+    _cuda(q, q_tail, k, v, k_tail, out, cu_q, kv_lens, gate)
+    _int32(cu_q, "cu_q")
+    _int32(kv_lens, "kv_lens")
+    rows = q.shape[0]
+    for name, t in (("q", q), ("k", k), ("v", v), ("out", out)):
+        _columns(t, name)
+        if t.dtype != torch.bfloat16 or t.shape[0] != rows:
+            raise KernelError(f"prompt_attention: {name} must be bfloat16 with {rows} rows, got {tuple(t.shape)} {t.dtype}")
+    key_dim, value_dim = k.shape[1] // heads, v.shape[1] // heads
+    if k.shape[1] != heads * key_dim or v.shape[1] != heads * value_dim or k.stride(0) != v.stride(0) or key_dim % 64 or value_dim % 64:
+        raise KernelError(f"prompt_attention: keys {tuple(k.shape)} and values {tuple(v.shape)} are no {heads} heads of whole 64 columns")
+    if out.shape[1] != heads * value_columns or value_columns > value_dim or q.shape[1] < heads * head_columns:
+        raise KernelError(f"prompt_attention: q {tuple(q.shape)} or out {tuple(out.shape)} does not fit {heads} heads")
+    turned = 0
+    if k_tail is not None:
+        turned = k_tail.shape[1]
+        if q_tail is None or tuple(k_tail.shape) != (rows, turned) or tuple(q_tail.shape) != (rows, heads * turned) \
+                or not k_tail.is_contiguous() or not q_tail.is_contiguous() or k_tail.dtype != q.dtype or q_tail.dtype != q.dtype:
+            raise KernelError("prompt_attention: shared key coordinates need contiguous [T, n] and [T, heads * n] rows")
+    if gate is not None:
+        _columns(gate, "gate")
+        if gate.dtype != q.dtype or tuple(gate.shape) != (rows, heads):
+            raise KernelError(f"prompt_attention: a gate per head cannot be {tuple(gate.shape)} {gate.dtype}")
+    lib = float_weight_attention_library(key_dim, value_dim, turned, True)
+    _run(lib, lib.mb_prompt_attention_tcgen05(
+        _p(q), q.stride(0), int(head_columns), q.shape[1], _p(q_tail), _p(k), _p(v), k.stride(0), _p(k_tail), rows, _p(out), out.stride(0),
+        int(value_columns), _p(gate), gate.stride(0) if gate is not None else 0, _p(cu_q), _p(kv_lens), kv_lens.numel(), int(max_q_len), heads,
+        heads, int(window), ctypes.c_float(scale), _stream()))
+
+
 def gated_decode_runs(sequences: int, heads: int, kv_heads: int, pages: int, multiprocessors: int = 148):
     """(runs, pages per run) for a decode step whose page tables are `pages` wide.  A block's four warps take a run's
     chunks of 32 keys in turn, and a warp's chunks cost it one wait for memory after another: runs of two pages (a chunk
@@ -859,12 +913,12 @@ def gated_attention(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, v_
     sequence's position 0; `window` n > 0: only if i - j < n.
     `kernel`: None picks the decode form for steps of one token per sequence (the keys cut into runs with a block each;
     the grid follows the page table's width, not the lengths, so that a captured step stays valid), the tensor-core form
-    where it applies (bfloat16 steps of many tokens), else the form with a warp per (token, head); decode steps of 8 heads and
-    more over rows they share run on the tensor cores, "tc_decode", where the sizes allow; "decode", "tc", "tc_decode" or "rows"
-    asks for one of them."""
+    where it applies (bfloat16 steps of many tokens; plain softmax attention of suitable sizes on the tcgen05 ones, "tcgen05"), else the form with a warp per (token, head); decode steps of 8 heads and
+    more over rows they share run on the tensor cores, "tc_decode", where the sizes allow; "decode", "tc", "tcgen05",
+    "tc_decode" or "rows" asks for one of them."""
     if weights not in ("softmax", "sigmoid"):
         raise KernelError(f"gated_attention: weights must be 'softmax' or 'sigmoid', got {weights!r}")
-    if kernel not in (None, "tc", "rows", "decode", "tc_decode"):
+    if kernel not in (None, "tc", "tcgen05", "rows", "decode", "tc_decode"):
         raise KernelError(f"gated_attention: unknown kernel {kernel!r}")
     if gate_kind not in GATE_KINDS or (gate_kind is None) != (gate is None):
         raise KernelError(f"gated_attention: gate kind {gate_kind!r} does not fit the gate given")
@@ -951,6 +1005,16 @@ def gated_attention(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, v_
             heads, kv_heads, head_dim, value_dim, page_size, softmax, ctypes.c_float(scale), ctypes.c_float(slope_exponent), runs,
             span, _p(scratch), *extras, _stream()))
         _launches[0] += 1  # two kernels
+        return
+    plain = plain_scores and weights == "softmax" and not sink and gate is None and block == 0
+    if kernel == "tcgen05" or (kernel is None and plain and float_weight_attention_takes(q, out, k_pool, v_pool, head_dim, value_dim, max_q_len)):
+        if not plain or not float_weight_attention_takes(q, out, k_pool, v_pool, head_dim, value_dim, max(max_q_len, TCGEN05_ATTENTION_MIN_ROWS)):
+            raise KernelError("the tcgen05 form takes plain softmax attention in bfloat16, pages of 64, and sizes that are multiples of 64")
+        lib = float_weight_attention_library(head_dim, value_dim)
+        _run(lib, lib.mb_prefill_attention_tcgen05(
+            _p(q), q.stride(0), q.shape[0], _p(out), out.stride(0), _p(k_pool), _p(v_pool), k_pool.shape[0], _p(block_table),
+            block_table.shape[1], _p(cu_q), _p(kv_lens), sequences, max_q_len, heads, kv_heads, page_size, int(window), ctypes.c_float(scale),
+            _stream()))
         return
     if kernel == "tc" or (kernel is None and gated_attention_tc_takes(q, out, k_pool, head_dim, value_dim, max_q_len, gate, gate_kind, v_pool)):
         if not gated_attention_tc_takes(q, out, k_pool, head_dim, value_dim, max(max_q_len, GATED_TC_MIN_ROWS), gate, gate_kind, v_pool):
@@ -1042,6 +1106,44 @@ def latent_prepare(q: Optional[torch.Tensor], q_gain: Optional[torch.Tensor], q_
                                     _p(cos) if turned else None, _p(sin) if turned else None, _p(positions), ctypes.c_float(eps),
                                     _p(k_pool) if k is not None else None, _p(slot_mapping), _code(dtype), rows, _stream()))
     return out
+
+
+def latent_rows(k: torch.Tensor, gain: torch.Tensor, turned: int, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor],
+                positions: torch.Tensor, eps: float, k_pool: torch.Tensor, slot_mapping: torch.Tensor, q: Optional[torch.Tensor] = None,
+                heads: int = 0, head_columns: int = 0, padded: int = 0):
+    """The cached rows of a latent attention whose queries have no latent of their own: k [T, latent + turned], the latent / rms * gain and
+    the tail rotated by the token's position (pairs (i, i + turned / 2), float32 tables [positions, turned / 2]), go into the pool
+    [pages, 1, page_size, latent + turned] at `slot_mapping`.  With `q` (a prompt that reads its own rows): also returns, in the step's
+    order, the latents [T, latent], the tails [T, padded] and the query heads' rotated tails [T, heads * padded], zeros behind
+    the `turned` numbers (None, None without a tail); head h's tail ends at column (h + 1) * head_columns of q."""
+    _cuda(k, gain, cos, sin, positions, k_pool, slot_mapping, q)
+    _int32(positions, "positions")
+    _int32(slot_mapping, "slot_mapping")
+    _columns(k, "k")
+    rows, latent = k.shape[0], k.shape[1] - turned
+    if gain.dtype != torch.float32 or gain.numel() != latent or not gain.is_contiguous():
+        raise KernelError(f"latent_rows: rows {tuple(k.shape)} with a tail of {turned} do not fit the gain")
+    if k_pool.dim() != 4 or k_pool.shape[1] != 1 or k_pool.shape[3] != k.shape[1] or not k_pool.is_contiguous() or k_pool.dtype != k.dtype:
+        raise KernelError(f"latent_rows: the pool must be contiguous [pages, 1, page_size, {k.shape[1]}] of {k.dtype}")
+    if turned:
+        for table in (cos, sin):
+            if table is None or table.dtype != torch.float32 or table.dim() != 2 or table.shape[1] * 2 != turned or not table.is_contiguous():
+                raise KernelError(f"latent_rows: a tail of {turned} needs contiguous float32 tables [positions, {turned // 2}]")
+    own = tail = q_tail = None
+    if q is not None:
+        _columns(q, "q")
+        if q.dtype != k.dtype or q.shape[0] != rows or q.shape[1] < heads * head_columns or head_columns < turned or padded < turned:
+            raise KernelError(f"latent_rows: queries {tuple(q.shape)} {q.dtype} are no {heads} heads of {head_columns}")
+        own = torch.empty((rows, latent), dtype=k.dtype, device=k.device)
+        if turned:
+            tail = torch.empty((rows, padded), dtype=k.dtype, device=k.device)
+            q_tail = torch.empty((rows, heads * padded), dtype=k.dtype, device=k.device)
+    lib = gated_attention_library()
+    _run(lib, lib.mb_latent_rows(_p(k), k.stride(0), _p(gain), latent, int(turned), _p(cos) if turned else None, _p(sin) if turned else None,
+                                 _p(positions), ctypes.c_float(eps), _p(k_pool), _p(slot_mapping), _p(own), _p(tail), _p(q),
+                                 q.stride(0) if q is not None else 0, head_columns - turned, heads, _p(q_tail), int(padded), _code(k.dtype), rows,
+                                 _stream()))
+    return own, tail, q_tail
 
 
 RETENTION_RUN = 64  # tokens of a run when a long step's recurrence is walked in runs

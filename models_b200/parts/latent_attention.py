@@ -4,8 +4,8 @@ q = Wq.xn (heads of `head_dim`); c = rmsnorm(Wd.xn) with a gain, `latent_dim` nu
 (one "key head" of latent_dim, no values).  Head h has k_j = Uk_h.c_j and v_j = Uv_h.c_j, so its score
 scale * q_i.k_j equals scale * (Uk_h^T q_i).c_j and its result sum_j w_j v_j equals Uv_h.(sum_j w_j c_j): the query is taken
 into the latent space once per token and head, the attention runs over the cached rows themselves (all heads read the same
-rows, as key and as value), and the result is taken out of the latent space once per token and head.  No key or value is
-ever expanded.  With `gated`, head h's result is multiplied by sigmoid((Wg.xn)_h); then Wo.  The
+rows, as key and as value), and the result is taken out of the latent space once per token and head.  No key or value of
+the cache is ever expanded.  With `gated`, head h's result is multiplied by sigmoid((Wg.xn)_h); then Wo.  The
 norm, the scores and the softmax are float32 in both modes.
 
 Variations (the spec says which).  Queries from a latent of their own, q = Uq.rmsnorm(Wdq.xn).  A position: every query head has
@@ -14,6 +14,10 @@ space is [Uk_h^T q | rotated part], the cached row [c | rotated part], and their
 row's first latent_dim numbers.  (Rotated pairs (2i, 2i + 1) are brought side by side when the weights are loaded: the rotated
 parts meet in dot products only, so the order of their coordinates is nobody's business but theirs, and the kernels know one
 pairing.)  A window.  A gate per element.  Rows that another run cached (`own_rows` False).
+
+A prompt that starts its sequences sees no row but its own, and there the other order is cheaper: one product expands every row of
+the step into the heads' keys and values, and the attention runs over those (with the shared rotated part beside them), a third of the
+multiplications per query and key.  Steps that continue a sequence, and sizes the kernel does not take, stay in the latent space.
 """
 
 from __future__ import annotations
@@ -27,6 +31,11 @@ from .base import Mixer, RunContext
 from .linear import linear, stack_columns, stack_rows
 from .registry import build_part, register_part
 from .split import SplitPart
+
+
+def _whole(size: int) -> int:
+    """The next multiple of 64: the columns of a shared-memory tile."""
+    return -(-size // 64) * 64
 
 
 class LatentAttentionMixer(SplitPart, Mixer):
@@ -96,6 +105,15 @@ class LatentAttentionMixer(SplitPart, Mixer):
         self.into_latent = rt.matrix(tensors[n["up_k"]]).to(dtype).view(s.num_heads, s.head_dim, s.latent_dim).transpose(1, 2).contiguous()
         self.out_of_latent = rt.matrix(tensors[n["up_v"]]).to(dtype).view(s.num_heads, s.value_dim, s.latent_dim).contiguous()
 
+        self.expand = None
+        K, D, V = s.latent_dim, s.head_dim, s.value_dim
+        if (rt.mode == "bfloat16" and s.own_rows and not s.query_latent and (not s.gated or s.gate_kind == "head") and K % 8 == 0
+                and (D + self.turned) % 8 == 0 and V % 8 == 0 and V <= 128 and _whole(D) + _whole(self.turned) <= 256):
+            # every head's key and value matrices padded with zero rows to whole 64s: [heads * keys; heads * values] x latent
+            pad = lambda m, size: torch.nn.functional.pad(m, (0, 0, 0, _whole(size) - size)).reshape(-1, K)  # noqa: E731
+            self.expand = torch.cat([pad(rt.matrix(tensors[n["up_k"]]).to(dtype).view(s.num_heads, D, K), D),
+                                     pad(self.out_of_latent, V)]).contiguous()
+
     def input_matrix(self):
         return self.w_in
 
@@ -119,7 +137,20 @@ class LatentAttentionMixer(SplitPart, Mixer):
         cos, sin = (self.rope.cos, self.rope.sin) if self.rope is not None else (None, None)
         down_q, down, gate = part("down_q"), part("down"), part("gate")
         q_rows = None
-        if down_q is not None or down is not None:
+        if down_q is None and down is not None:
+            q = part("q")
+            fresh = (self.expand is not None and getattr(batch, "fresh", False) and batch.max_q_len >= ops.TCGEN05_ATTENTION_MIN_ROWS
+                     and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and mid.stride(0) % 8 == 0 and mid.data_ptr() % 16 == 0)
+            more = {"q": q, "heads": s.num_heads, "head_columns": s.head_dim + self.turned, "padded": _whole(self.turned)} if fresh else {}
+            own, tail, q_tail = ops.latent_rows(down, self.latent_gain, self.turned, cos, sin, batch.positions, s.eps, run.k_pool,
+                                                group.slot_mapping, **more)
+            if fresh:
+                at = s.num_heads * _whole(s.head_dim)
+                expanded = linear(own, self.expand, own.dtype)
+                ops.prompt_attention(q, q_tail, expanded[:, :at], expanded[:, at:], tail, mid, batch.cu_q, batch.kv_lens, batch.max_q_len,
+                                     s.num_heads, s.head_dim + self.turned, s.value_dim, s.scale, gate, s.window or 0)
+                return
+        elif down_q is not None:
             q_rows = ops.latent_prepare(down_q, self.query_gain if down_q is not None else None, self.up_q.shape[1] if down_q is not None else 0,
                                         down, self.latent_gain, self.turned, cos, sin, batch.positions, s.eps, run.k_pool, group.slot_mapping)
         q = part("q") if down_q is None else linear(q_rows, self.up_q, proj.dtype)

@@ -248,11 +248,102 @@ def _run_in_pieces(part, h, cuts, dtype, device):
                     table[0, block] = 0
         batch = SimpleNamespace(positions=positions[at:at + n].contiguous(), cu_q=torch.tensor([0, n], dtype=torch.int32, device=device),
                                 kv_lens=torch.tensor([at + n], dtype=torch.int32, device=device), max_q_len=n,
-                                groups=[SimpleNamespace(block_table=table, slot_mapping=mapping[at:at + n].contiguous())])
+                                fresh=at == 0, groups=[SimpleNamespace(block_table=table, slot_mapping=mapping[at:at + n].contiguous())])
         run = SimpleNamespace(group=0, k_pool=k_pool, v_pool=v_pool, writes_cache=True)
         rows.append(part.forward(h[at:at + n].to(td).to(device), batch, run).float().cpu())
         at += n
     return torch.cat(rows)
+
+
+@pytest.mark.parametrize("heads,kv_heads,dim,value_dim", [(4, 2, 128, 128), (3, 1, 64, 64), (2, 2, 64, 128), (2, 1, 192, 128), (2, 2, 256, 64)])
+@pytest.mark.parametrize("window", [None, 1, 64, 65, 130])
+def test_prompt_attention_on_pages_unequal_and_continued(cuda_device, heads, kv_heads, dim, value_dim, window):
+    """The tcgen05 form with float weights over pages full of NaN where nothing was written: a batch of prompts of unequal lengths, one
+    of which goes on where earlier steps left it; loud keys that move the running maximum late."""
+    from models_b200.kernels import ops
+
+    g = torch.Generator().manual_seed(dim + (window or 0))
+    lengths, counts = [300, 64, 1, 129, 200], [300, 64, 1, 129, 70]
+    bf = torch.bfloat16
+    pages = [-(-n // 64) for n in lengths]
+    table = torch.zeros((len(lengths), max(pages)), dtype=torch.int32)
+    order = (torch.randperm(sum(pages), generator=g) + 1).to(torch.int32)
+    at = 0
+    for i, n in enumerate(pages):
+        table[i, :n] = order[at:at + n]
+        at += n
+    k_pool = torch.full((at + 1, kv_heads, 64, dim), float("nan"), dtype=bf, device=cuda_device)
+    v_pool = torch.full((at + 1, kv_heads, 64, value_dim), float("nan"), dtype=bf, device=cuda_device)
+    scale, wants, qs = 0.6 * dim ** -0.5, [], []
+    for i, (n, count) in enumerate(zip(lengths, counts)):
+        q, k, v = (_rounded(torch.randn(n, h, size, generator=g) * a, bf) for h, size, a in ((heads, dim, 1.0), (kv_heads, dim, 1.5), (kv_heads, value_dim, 1.0)))
+        k[n // 2] *= 8.0  # (exact in bfloat16)
+        for p in range(n):
+            k_pool[table[i, p // 64], :, p % 64] = k[p].to(bf).to(cuda_device)
+            v_pool[table[i, p // 64], :, p % 64] = v[p].to(bf).to(cuda_device)
+        seen = pr.window_visible(n, window)
+        want = torch.stack([pr.softmax_sum(q[:, h] @ k[:, h * kv_heads // heads].T * scale, seen, v[:, h * kv_heads // heads]) for h in range(heads)], 1)
+        wants.append(want[n - count:].reshape(count, -1))
+        qs.append(q[n - count:].reshape(count, -1))
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=cuda_device)  # noqa: E731
+    rows = torch.cat(qs).to(bf).to(cuda_device)
+    out = torch.full((rows.shape[0], heads * value_dim), float("nan"), dtype=bf, device=cuda_device)
+    cu = i32(np.concatenate([[0], np.cumsum(counts)]).tolist())
+    ops.gated_attention(rows, out, k_pool, v_pool, table.to(cuda_device), cu, i32(lengths), max(counts), heads, kv_heads, dim, value_dim, "softmax",
+                        scale, window=window or 0, kernel="tcgen05")
+    assert scaled_error(out.double().cpu(), torch.cat(wants)) < 6e-3
+    other = torch.empty_like(out)
+    ops.gated_attention(rows, other, k_pool, v_pool, table.to(cuda_device), cu, i32(lengths), max(counts), heads, kv_heads, dim, value_dim, "softmax",
+                        scale, window=window or 0, kernel="rows")
+    assert scaled_error(out.double().cpu(), other.double().cpu()) < 6e-3
+
+
+@pytest.mark.parametrize("heads,dim,rot,value_dim,gated", [(3, 64, 64, 128, True), (2, 48, 16, 40, True), (4, 64, 0, 64, False), (1, 128, 64, 128, True),
+                                                           (2, 8, 8, 8, True), (2, 96, 104, 72, False)])
+def test_prompt_attention_on_its_own_rows(cuda_device, heads, dim, rot, value_dim, gated):
+    """Prompts of unequal lengths that start their sequences; rows behind the last sequence hold NaN (they belong to nobody), columns of
+    padding hold zeros in keys and values and anything finite in the queries; a gate per head."""
+    from models_b200.kernels import ops
+
+    g = torch.Generator().manual_seed(dim + rot)
+    whole = lambda n: -(-n // 64) * 64  # noqa: E731
+    bf, lengths = torch.bfloat16, [70, 1, 300, 64, 33]
+    T = sum(lengths)
+    spare = 20
+    KD, RD, VD = whole(dim), whole(rot), whole(value_dim)
+    scale = 1.3 * (dim + rot) ** -0.5
+    q = _rounded(torch.randn(T, heads, dim + rot, generator=g), bf)
+    k, v, r = (_rounded(torch.randn(*s, generator=g), bf) for s in ((T, heads, dim), (T, heads, value_dim), (T, rot)))
+    gate = _rounded(torch.randn(T, heads, generator=g), bf)
+    wants, at = [], 0
+    for n in lengths:
+        s = slice(at, at + n)
+        score = [(q[s, h, :dim] @ k[s, h].T + q[s, h, dim:] @ r[s].T) * scale for h in range(heads)]
+        one = torch.stack([pr.softmax_sum(score[h], pr.window_visible(n, None), v[s, h]) for h in range(heads)], 1)
+        wants.append((one * torch.sigmoid(gate[s])[:, :, None] if gated else one).reshape(n, -1))
+        at += n
+    nan = lambda *shape: torch.full(shape, float("nan"), dtype=bf, device=cuda_device)  # noqa: E731
+
+    def rows(t, size, heads=heads):  # [T, heads, n] -> [T + spare, heads * size], zeros in the padding, NaN behind
+        out = nan(T + spare, heads * size)
+        padded = torch.zeros(T, heads, size, dtype=F)
+        padded[:, :, :t.shape[-1]] = t
+        out[:T] = padded.reshape(T, -1).to(bf).to(cuda_device)
+        return out
+
+    kv = torch.cat([rows(k, KD), rows(v, VD)], dim=1).contiguous()
+    q_rows = nan(T + spare, heads * (dim + rot))
+    q_rows[:T] = q.reshape(T, -1).to(bf).to(cuda_device)
+    out = torch.full((T + spare, heads * value_dim + 8), 7.0, dtype=bf, device=cuda_device)
+    gates = nan(T + spare, heads)
+    gates[:T] = gate.to(bf).to(cuda_device)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=cuda_device)  # noqa: E731
+    ops.prompt_attention(q_rows, rows(q[..., dim:], RD) if rot else None, kv[:, :heads * KD], kv[:, heads * KD:],
+                         rows(r[:, None], RD, 1) if rot else None, out[:, :heads * value_dim],
+                         i32(np.concatenate([[0], np.cumsum(lengths)]).tolist()), i32(lengths), max(lengths), heads, dim + rot, value_dim, scale,
+                         gates if gated else None)
+    assert scaled_error(out[:T, :heads * value_dim].double().cpu(), torch.cat(wants)) < 6e-3
+    assert bool((out[T:] == 7).all()) and bool((out[:, heads * value_dim:] == 7).all())
 
 
 CUTS = ([200], [2, 60, 1, 77, 60], [70] + [1] * 130)
