@@ -1287,24 +1287,43 @@ def rulunex_kernels(z, peak, prompt=2048, batch=8, context=1536):
         pages = sequences * (-(-lengths[0] // page))
         table = (torch.arange(pages, dtype=torch.int32, device=dev) + 1).reshape(sequences, -1).contiguous()
         mapping = (torch.arange(rows, dtype=torch.int32, device=dev) + page)
-        # latent attention over every earlier position, a gate per head; beside Mabivik's (a window, a query latent, gates per element)
+        # latent attention over every earlier position, a gate per head: a starting prompt's rows expanded by one product, decoding over
+        # the cached rows; beside Mabivik's over the cached rows (a window, a query latent, gates per element)
         pool = low(pages + 1, 1, page, K + R)
         q, o = low(rows, LH * (K + R)), torch.empty((rows, LH * K), dtype=bf, device=dev)
         for title, win, used in (("latent_attention", 0, all_pairs), ("latent_attention_mabivik", window, windowed)):
+            if q_len > 1 and not win:
+                continue
             us = time_kernel(lambda: ops.gated_attention(q, o, pool, None, table, cu, kv, q_len, LH, 1, K + R, K, "softmax", LD ** -0.5, window=win))
             out[f"{name}_{title}"] = rated(us, flops=used * LH * (2 * (K + R) + 2 * K)) if q_len > 1 else \
                 rated(us, moved=sum(min(n, win or n) for n in lengths) * (K + R) * 2)
         x, y = low(rows, LH * (LD + R)), torch.empty((rows, LH * DV), dtype=bf, device=dev)
         into, outof = low(LH, K, LD), low(LH, DV, K)
-        for title, gate, kind in (("head_products", low(rows, LH), "head"), ("head_products_mabivik", low(rows, LH * DV), "element")):
+        gate = low(rows, LH)
+        if q_len > 1:
+            KD, VD, RD = (-(-n // 64) * 64 for n in (LD, DV, R))
+            own, expand = low(rows, K), low(LH * (KD + VD), K)
+            us = time_kernel(lambda: linear(own, expand, bf))
+            out["prompt_latent_expansion"] = rated(us, flops=rows * LH * 2 * K * (LD + DV))
+            wide, tail, q_tail = low(rows, LH * (KD + VD)), low(rows, RD), low(rows, LH * RD)
+            us = time_kernel(lambda: ops.prompt_attention(x, q_tail, wide[:, :LH * KD], wide[:, LH * KD:], tail, y, cu, kv, q_len, LH, LD + R, DV,
+                                                          LD ** -0.5, gate))
+            out["prompt_latent_attention"] = rated(us, flops=all_pairs * LH * 2 * (LD + R + DV))
+        for title, gate, kind in (("head_products", gate, "head"), ("head_products_mabivik", low(rows, LH * DV), "element")):
+            if q_len > 1 and kind == "head":
+                continue
             us = time_kernel(lambda: (ops.head_linear(x, into, q, LH, turned=R, cos=cos, sin=sin, positions=positions),
                                       ops.head_linear(o, outof, y, LH, gate, gate_kind=kind)))
             out[f"{name}_{title}"] = rated(us, flops=rows * LH * 2 * K * (LD + DV)) if q_len > 1 else \
                 rated(us, moved=LH * K * (LD + DV) * 2 + rows * LH * (LD + K + K + DV) * 2)
         Q = K * 2
         first, gq, gk = low(rows, Q + K + R), torch.ones(Q, device=dev), torch.ones(K, device=dev)
-        us = time_kernel(lambda: ops.latent_prepare(None, None, 0, first[:, Q:], gk, R, cos, sin, positions, 1e-6, pool, mapping))
-        out[f"{name}_latent_prepare"] = rated(us, moved=rows * 4 * (K + R))
+        if q_len > 1:  # with the rows in the step's order and the queries' rotated parts
+            us = time_kernel(lambda: ops.latent_rows(first[:, Q:], gk, R, cos, sin, positions, 1e-6, pool, mapping, q=x, heads=LH, head_columns=LD + R, padded=RD))
+            out["prompt_latent_rows"] = rated(us, moved=rows * (6 * (K + R) + 4 * LH * R))
+        else:
+            us = time_kernel(lambda: ops.latent_rows(first[:, Q:], gk, R, cos, sin, positions, 1e-6, pool, mapping))
+            out["decode_latent_rows"] = rated(us, moved=rows * 4 * (K + R))
         us = time_kernel(lambda: ops.latent_prepare(first[:, :Q], gq, Q, first[:, Q:], gk, R, cos, sin, positions, 1e-6, pool, mapping))
         out[f"{name}_latent_prepare_mabivik"] = rated(us, moved=rows * 4 * (Q + K + R))
         # windowed attention with the projected keys as values; beside Rolevik's over chunks as long as the window, values of their own

@@ -246,8 +246,10 @@ class PromptGraphs:
     def __init__(self, decode_graphs: DecodeGraphs):
         self.decode_graphs = decode_graphs
         self.engine = decode_graphs.engine
-        self.captured: Dict[tuple, _Captured] = {}  # (batch size, token count, page-table width, whether the sequences start)
+        self.captured: Dict[tuple, _Captured] = {}  # (batch size, token count, page-table width[, whether the sequences start])
         self.uses: Dict[tuple, int] = {}
+        # whether some mixer's launches differ for prompts that start their sequences: their class then says so
+        self.by_start = any(getattr(block.mixer, "starts_differ", False) for block in self.engine.model.blocks)
 
     def bucket(self, entries: Sequence) -> Optional[tuple]:
         """The class of the step, or None for one that runs launch by launch: too many tokens or
@@ -263,7 +265,8 @@ class PromptGraphs:
         longest = max(cache.lengths[slot] + len(tokens) for slot, tokens, _ in entries)
         if -(-longest // cache.page_size) > graphs.blocks:
             return None
-        return size, next(t for t in PROMPT_TOKENS if t >= total), graphs.table_width(longest), starts_sequences(cache, entries)
+        key = size, next(t for t in PROMPT_TOKENS if t >= total), graphs.table_width(longest)
+        return key + (starts_sequences(cache, entries),) if self.by_start else key
 
     def step(self, entries: Sequence) -> Optional[torch.Tensor]:
         """entries: (slot, tokens, wanted places); the cache already has room.  Returns the logits of
@@ -278,7 +281,7 @@ class PromptGraphs:
             if self.uses[key] <= EAGER_USES or len(self.captured) >= MAX_PROMPT_CAPTURES:
                 return None
             graphs = self.decode_graphs
-            captured = self.captured[key] = _Captured(self.engine, key[0], key[2], graphs.pool, tokens=key[1], fresh=key[3])
+            captured = self.captured[key] = _Captured(self.engine, key[0], key[2], graphs.pool, tokens=key[1], fresh=self.by_start and key[3])
         wanted = captured.fill(self.engine.cache, entries)
         captured.upload()
         captured.graph.replay()

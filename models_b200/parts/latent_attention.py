@@ -114,6 +114,11 @@ class LatentAttentionMixer(SplitPart, Mixer):
             self.expand = torch.cat([pad(rt.matrix(tensors[n["up_k"]]).to(dtype).view(s.num_heads, D, K), D),
                                      pad(self.out_of_latent, V)]).contiguous()
 
+    @property
+    def starts_differ(self) -> bool:
+        """Whether prompts that start their sequences take another way than steps that continue them."""
+        return getattr(self, "expand", None) is not None
+
     def input_matrix(self):
         return self.w_in
 
