@@ -1576,7 +1576,16 @@ MB_EXPORT int mb_project_norm_rotate_store(void* q, int q_stride, const void* k,
     if (tokens <= 0) return 0;
     if (rotary_dim < 0 || rotary_dim % 2 || rotary_dim > head_dim) return fail("project_norm_rotate_store: rotary_dim %d of heads of %d", rotary_dim, head_dim);
     const size_t smem = sizeof(float) * (size_t)(heads + kv_heads) * head_dim;
-    if (smem > 40 * 1024) return fail("project_norm_rotate_store: rows of %d numbers exceed the 10240 a block keeps", (heads + kv_heads) * head_dim);
+    if (smem > 200 * 1024) return fail("project_norm_rotate_store: rows of %d numbers exceed the 51200 a block keeps", (heads + kv_heads) * head_dim);
+    if (smem > 40 * 1024) {  // (beside the static scratch)
+        const void* kernels[] = {(const void*)project_norm_rotate_store_kernel<float>, (const void*)project_norm_rotate_store_kernel<__nv_bfloat16>,
+                                 (const void*)project_norm_rotate_store_vec8_kernel<float>,
+                                 (const void*)project_norm_rotate_store_vec8_kernel<__nv_bfloat16>};
+        for (const void* kernel : kernels) {
+            cudaError_t status = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            if (status != cudaSuccess) return fail("project_norm_rotate_store: cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(status));
+        }
+    }
     const Rotation rotation{cos, sin, rotary_dim, interleaved, 0, nullptr, nullptr, 0};
     const size_t element = dtype == MB_F32 ? 4 : 2, row_bytes = 8 * element - 1;
     const bool wide = head_dim % 8 == 0 && value_dim % 8 == 0 && rotary_dim % (interleaved ? 8 : 16) == 0 && q_stride % 8 == 0 && k_stride % 8 == 0 &&

@@ -346,6 +346,86 @@ def test_prompt_attention_on_its_own_rows(cuda_device, heads, dim, rot, value_di
     assert bool((out[T:] == 7).all()) and bool((out[:, heads * value_dim:] == 7).all())
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("heads,kv_heads,dim,rot,interleaved", [(20, 4, 128, 64, False), (96, 16, 128, 128, False), (3, 1, 24, 8, True), (5, 5, 10, 6, False),
+                                                                (4, 2, 16, 16, True), (2, 1, 40, 0, False), (6, 3, 32, 8, False)])
+def test_whole_projections_normed_rotated_and_stored(cuda_device, heads, kv_heads, dim, rot, interleaved, dtype):
+    """The kernel alone, in its wide and its element-wise form, up to rows of 14,336 numbers; the values are the keys' own columns."""
+    from models_b200.kernels import ops
+
+    g = torch.Generator().manual_seed(heads)
+    td, T, q_width, k_width = TORCH[dtype], 5, heads * dim, kv_heads * dim
+    rows = _rounded(torch.randn(T, q_width + k_width, generator=g) * torch.tensor([0.1, 1.0, 3.0, 1.0, 0.5])[:, None], td)
+    gains = 1 + 0.3 * torch.randn(q_width + k_width, generator=g)
+    positions = torch.tensor([0, 1, 70, 5, 300])
+    angle = positions.double()[:, None] * torch.tensor([50.0 ** (-2.0 * i / max(rot, 1)) for i in range(rot // 2)], dtype=F)[None, :]
+    table = torch.arange(301).double()[:, None] * torch.tensor([50.0 ** (-2.0 * i / max(rot, 1)) for i in range(rot // 2)], dtype=F)[None, :]
+    cos, sin = (f(table).float().contiguous().to(cuda_device) if rot else None for f in (torch.cos, torch.sin))
+
+    def expected(x, gain, count):
+        y = (pr.over_rms(x, 1e-4) * gain.double()).view(T, count, dim)
+        c, s = torch.cos(angle)[:, None], torch.sin(angle)[:, None]
+        u, v = (y[..., 0:rot:2], y[..., 1:rot:2]) if interleaved else (y[..., :rot // 2], y[..., rot // 2:rot])
+        a, b = u * c - v * s, v * c + u * s
+        turned = torch.stack([a, b], -1).flatten(-2) if interleaved else torch.cat([a, b], -1)
+        return torch.cat([turned, y[..., rot:]], -1)
+
+    proj = rows.to(td).to(cuda_device)
+    pools = [torch.full((3, kv_heads, 64, dim), float("nan"), dtype=td, device=cuda_device) for _ in range(2)]
+    slots = torch.tensor([70, 64, -1, 191, 130], dtype=torch.int32, device=cuda_device)  # (the third token stores nothing)
+    q, k = proj[:, :q_width], proj[:, q_width:]
+    ops.project_norm_rotate_store(q, k, k, None, None, None, gains[:q_width].to(cuda_device).contiguous(), gains[q_width:].to(cuda_device).contiguous(), 1e-4,
+                                  positions.to(torch.int32).to(cuda_device), cos, sin, rot, interleaved, pools[0], pools[1], slots, heads, kv_heads, dim, dim)
+    bound = 2e-6 if dtype == "float32" else 5e-3
+    assert scaled_error(proj[:, :q_width].double().cpu().view(T, heads, dim), expected(rows[:, :q_width], gains[:q_width], heads)) < bound
+    want = expected(rows[:, q_width:], gains[q_width:], kv_heads)
+    raw = rows[:, q_width:].view(T, kv_heads, dim)
+    for i, slot in enumerate(slots.tolist()):
+        if slot >= 0:
+            for pool, w in zip(pools, (want[i], raw[i])):
+                assert scaled_error(pool[slot // 64, :, slot % 64].double().cpu(), w) < bound
+    assert int(torch.isnan(pools[0]).any(-1).sum()) == int(torch.isnan(pools[1]).any(-1).sum()) == kv_heads * (3 * 64 - 4)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("latent_dim,turned,heads,dim", [(256, 64, 4, 64), (64, 16, 3, 48), (26, 6, 2, 10), (320, 0, 2, 64), (40, 8, 5, 8), (9, 2, 1, 6)])
+def test_latent_rows_for_the_cache_and_for_the_step(cuda_device, latent_dim, turned, heads, dim, dtype):
+    from models_b200.kernels import ops
+
+    g = torch.Generator().manual_seed(latent_dim)
+    td, T, padded = TORCH[dtype], 4, -(-turned // 64) * 64
+    k, q = _rounded(torch.randn(T, latent_dim + turned, generator=g), td), _rounded(torch.randn(T, heads * (dim + turned), generator=g), td)
+    gain, positions = 1 + 0.3 * torch.randn(latent_dim, generator=g), torch.tensor([3, 0, 90, 17])
+    table = torch.arange(100).double()[:, None] * torch.tensor([30.0 ** (-2.0 * i / max(turned, 1)) for i in range(turned // 2)], dtype=F)[None, :]
+    c, s = torch.cos(table)[positions], torch.sin(table)[positions]
+
+    def rotated(x):  # pairs (i, i + turned / 2)
+        u, v = x[..., :turned // 2], x[..., turned // 2:]
+        cc, ss = (c, s) if x.dim() == 2 else (c[:, None], s[:, None])
+        return torch.cat([u * cc - v * ss, v * cc + u * ss], -1)
+
+    latent = pr.over_rms(k[:, :latent_dim], 1e-4) * gain.double()
+    tail, q_tail = rotated(k[:, latent_dim:]), rotated(q.view(T, heads, dim + turned)[..., dim:])
+    bound = 2e-6 if dtype == "float32" else 5e-3
+    dev = lambda t: t.to(td).to(cuda_device)  # noqa: E731
+    tables = tuple(f(table).float().contiguous().to(cuda_device) if turned else None for f in (torch.cos, torch.sin))
+    for queries in (None, dev(q)):
+        pool = torch.full((2, 1, 64, latent_dim + turned), float("nan"), dtype=td, device=cuda_device)
+        slots = torch.tensor([65, -1, 0, 127], dtype=torch.int32, device=cuda_device)
+        more = {} if queries is None else {"q": queries, "heads": heads, "head_columns": dim + turned, "padded": padded}
+        own, own_tail, own_q = ops.latent_rows(dev(k), gain.to(cuda_device), turned, *tables, positions.to(torch.int32).to(cuda_device), 1e-4, pool, slots, **more)
+        for i, slot in enumerate(slots.tolist()):
+            if slot >= 0:
+                assert scaled_error(pool.view(-1, latent_dim + turned)[slot].double().cpu(), torch.cat([latent[i], tail[i]])) < bound
+        assert int(torch.isnan(pool).any(-1).sum()) == 2 * 64 - 3
+        if queries is not None:
+            assert scaled_error(own.double().cpu(), latent) < bound
+            if turned:
+                assert scaled_error(own_tail[:, :turned].double().cpu(), tail) < bound and bool((own_tail[:, turned:] == 0).all())
+                got = own_q.view(T, heads, padded)
+                assert scaled_error(got[..., :turned].double().cpu(), q_tail) < bound and bool((got[..., turned:] == 0).all())
+
+
 CUTS = ([200], [2, 60, 1, 77, 60], [70] + [1] * 130)
 MIXERS = {
     "latent-small": latent(4, 16, 8, 8, 32, 0.3, 10000.0, 0), "latent-cores": latent(2, 64, 16, 32, 112, 0.11, 20000.0, 0),

@@ -138,6 +138,19 @@ def test_rotation_tables(rot):
         assert s is not STRETCHED or dims < 64 or bool(((ratio < 0.999) & (ratio > 1.001 / s[0])).any())
 
 
+def test_random_weights_put_layer_norms_around_zero():
+    """A weight stored as its distance from one is drawn around zero, a plain one around one."""
+    from models_b200.config import config_from_dict
+    from models_b200.engine.model import parameter_requests
+    from models_b200.weights.random_init import random_tensors
+
+    t = random_tensors(parameter_requests(config_from_dict(RLX["C"]).model_spec()), 5, gain_std=0.1)
+    for name in ("l0.norm1", "l3.norm1", "final.norm"):
+        assert abs(float(t[name].float().mean())) < 0.05 and 0.05 < float(t[name].float().std()) < 0.15
+    for name in ("l1.mix.q.norm", "l1.mix.k.norm", "l0.mix.dkv.norm"):
+        assert abs(float(t[name].float().mean()) - 1.0) < 0.05
+
+
 # ----------------------------------------------------------------------------------- the plain implementation
 
 def test_plain_mechanisms_by_hand():
